@@ -1,4 +1,5 @@
 from .fields import read_config_dict, required, optional
+from .fumolorn import FumolornConfig
 from .mabedra import MabedraConfig
 from .qwen3 import Qwen3Config
 from .ropulix import RopulixConfig
@@ -14,6 +15,7 @@ from .registry import (
 
 __all__ = [
     "Architecture",
+    "FumolornConfig",
     "MabedraConfig",
     "Qwen3Config",
     "RopulixConfig",

@@ -7,7 +7,8 @@
 // Eight warps: warp w owns rows 16 (w & 3) .. + 15 and the value columns of half (w >> 2); both warps of a row group
 // form the same scores S = Q K^T (mma.sync m16n8k16, float accumulation), run the same online softmax in float32, round
 // P to bfloat16 and multiply it with their half of the value columns, read transposed out of the key tile.
-// Key t is visible to a query at position p iff t <= p and (window == 0 or t > p - window).
+// Key t is visible to a query at position p iff t <= p and (window == 0 or t > p - window).  With a sink every head's sum has
+// one more term exp(sink[head]), which belongs to no key.
 #include "common.cuh"
 #include "mma.cuh"
 
@@ -39,6 +40,7 @@ struct LatentParams {
   const int* tile_count;
   int table_stride, page_size, heads, group_heads, tokens_per_tile, window;
   float scale_log2;
+  const float* sink;        // [heads] or null
   // a tile's keys cut into `splits` parts (single tokens only): CTA z takes its share of the key tiles and leaves
   // (maximum, sum) and the unnormalised output of row token * heads + head in scratch memory for the merge kernel
   int splits;
@@ -120,6 +122,14 @@ latent_attention_kernel(const LatentParams p) {
 #pragma unroll
     for (int e = 0; e < 4; ++e) o[j][e] = 0.f;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  if (p.sink != nullptr && blockIdx.z == 0) {       // the first part of a token's keys holds the sink: it starts the maximum and sum
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+      if (row_head[i] < p.heads) {
+        m[i] = p.sink[row_head[i]] * 1.4426950408889634f;
+        l[i] = 1.f;
+      }
+  }
 
   for (int kt = 0; kt < tiles; ++kt) {
     const int t0 = t_begin + kt * BN;
@@ -267,7 +277,7 @@ extern "C" int b200_attention_latent_rot() { return LATENT_ROT; }
 // tokens of one entry, at most tokens_per_tile = max(1, 64 / heads) each.  splits > 1 (every tile is token t alone, tile t):
 // the keys of a token are cut into that many parts, merged by a second launch; scratch holds splits * (DV + 2) floats a row.
 extern "C" int b200_attention_latent_bf16(const void* q, const void* pool, void* out, const int* positions, const int* block_table,
-                                          int table_stride, int page_size, int heads, float scale, int window, const int* tile_entry,
+                                          int table_stride, int page_size, int heads, float scale, int window, const float* sink, const int* tile_entry,
                                           const int* tile_start, const int* tile_count, int num_tiles, int splits, float* scratch,
                                           long scratch_floats, cudaStream_t stream) {
   using namespace b200;
@@ -293,6 +303,7 @@ extern "C" int b200_attention_latent_bf16(const void* q, const void* pool, void*
   p.tokens_per_tile = BM / p.group_heads;
   p.window = window;
   p.scale_log2 = scale * 1.4426950408889634f;
+  p.sink = sink;
   p.splits = splits;
   if (splits > 1) {
     p.tokens_per_tile = 1;

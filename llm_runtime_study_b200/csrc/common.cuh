@@ -56,6 +56,14 @@ template <> struct Vec<__nv_bfloat16> {
   }
 };
 
+// A gated unit's gate: silu(g) = g / (1 + e^-g), or the tanh form of gelu, which is the same with another exponent:
+// 0.5 g (1 + tanh(w)) = g / (1 + e^(-2w)), w = sqrt(2 / pi) (g + 0.044715 g^3).
+enum GateAct : int { ACT_SILU = 1, ACT_GELU_TANH = 2 };
+__device__ __forceinline__ float gate_exponent(float g, int act) {
+  return act == ACT_GELU_TANH ? 1.5957691216057308f * fmaf(0.044715f * g * g, g, g) : g;
+}
+__device__ __forceinline__ float gate_act(float g, int act) { return g / (1.f + expf(-gate_exponent(g, act))); }
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -193,9 +193,9 @@ __global__ void add_rmsnorm_vec_kernel(float* __restrict__ resid, const float* _
   }
 }
 
-// ------------------------------------------------------------------ SiLU * up
+// ------------------------------------------------------------------ SiLU (or another gate of common.cuh) * up
 template <typename T>
-__global__ void silu_mul_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inter) {
+__global__ void silu_mul_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inter, int act) {
   pdl_trigger();
   pdl_wait();
   const size_t row = blockIdx.y;
@@ -203,13 +203,12 @@ __global__ void silu_mul_kernel(const T* __restrict__ gate_up, T* __restrict__ o
   if (i >= inter) return;
   const float g = to_float(gate_up[row * 2 * inter + i]);
   const float u = to_float(gate_up[row * 2 * inter + inter + i]);
-  const float s = g / (1.f + expf(-g));
-  out[row * inter + i] = from_float<T>(s * u);
+  out[row * inter + i] = from_float<T>(gate_act(g, act) * u);
 }
 
 // 16-byte loads and stores when the row width allows it
 template <typename T>
-__global__ void silu_mul_vec_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inter) {
+__global__ void silu_mul_vec_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inter, int act) {
   constexpr int VN = Vec<T>::n;
   using V = typename Vec<T>::type;
   pdl_trigger();
@@ -221,7 +220,7 @@ __global__ void silu_mul_vec_kernel(const T* __restrict__ gate_up, T* __restrict
   Vec<T>::unpack(*reinterpret_cast<const V*>(gate_up + row * 2 * inter + i), g);
   Vec<T>::unpack(*reinterpret_cast<const V*>(gate_up + row * 2 * inter + inter + i), u);
 #pragma unroll
-  for (int e = 0; e < VN; ++e) g[e] = g[e] / (1.f + expf(-g[e])) * u[e];
+  for (int e = 0; e < VN; ++e) g[e] = gate_act(g[e], act) * u[e];
   *reinterpret_cast<V*>(out + row * inter + i) = Vec<T>::pack(g);
 }
 
@@ -322,7 +321,7 @@ __global__ void __launch_bounds__(kRopeWarps * 32) qk_norm_rope_write_kernel(
 // the layout in which the stacked gate/up projection is stored so that a projection kernel
 // can apply SiLU * up in its epilogue.  `inter` is a multiple of 8.
 template <typename T>
-__global__ void silu_mul_interleaved_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inter) {
+__global__ void silu_mul_interleaved_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int inter, int act) {
   pdl_trigger();
   pdl_wait();
   const size_t row = blockIdx.y;
@@ -339,7 +338,7 @@ __global__ void silu_mul_interleaved_kernel(const T* __restrict__ gate_up, T* __
     Vec<T>::unpack(*reinterpret_cast<const V*>(src + 8 + i), u + i);
   }
 #pragma unroll
-  for (int i = 0; i < 8; ++i) g[i] = g[i] / (1.f + expf(-g[i])) * u[i];
+  for (int i = 0; i < 8; ++i) g[i] = gate_act(g[i], act) * u[i];
 #pragma unroll
   for (int i = 0; i < 8; i += VN) *reinterpret_cast<V*>(dst + i) = Vec<T>::pack(g + i);
 }
@@ -619,34 +618,34 @@ extern "C" int b200_add_rmsnorm(float* resid, const float* delta, const float* w
   return launch_status();
 }
 
-extern "C" int b200_silu_mul(const void* gate_up, void* out, int n, int inter, int dtype,
+extern "C" int b200_silu_mul(const void* gate_up, void* out, int n, int inter, int act, int dtype,
                              cudaStream_t stream) {
   if (n <= 0) return 0;
-  if (inter <= 0) return B200_ERR_BAD_SIZE;
+  if (inter <= 0 || (act != ACT_SILU && act != ACT_GELU_TANH)) return B200_ERR_BAD_SIZE;
   if (n > 65535) return B200_ERR_TOO_LARGE;
   B200_DISPATCH_DTYPE(dtype, T, {
     constexpr int VN = Vec<T>::n;
     const bool aligned = ((reinterpret_cast<uintptr_t>(gate_up) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
     if (inter % VN == 0 && aligned) {
       dim3 grid((inter / VN + 255) / 256, n);
-      launch(silu_mul_vec_kernel<T>, dim3(grid), dim3(256), 0, stream, static_cast<const T*>(gate_up), static_cast<T*>(out), inter);
+      launch(silu_mul_vec_kernel<T>, dim3(grid), dim3(256), 0, stream, static_cast<const T*>(gate_up), static_cast<T*>(out), inter, act);
     } else {
       dim3 grid((inter + 255) / 256, n);
-      launch(silu_mul_kernel<T>, dim3(grid), dim3(256), 0, stream, static_cast<const T*>(gate_up), static_cast<T*>(out), inter);
+      launch(silu_mul_kernel<T>, dim3(grid), dim3(256), 0, stream, static_cast<const T*>(gate_up), static_cast<T*>(out), inter, act);
     }
   });
   return launch_status();
 }
 
-extern "C" int b200_silu_mul_interleaved(const void* gate_up, void* out, int n, int inter, int dtype,
+extern "C" int b200_silu_mul_interleaved(const void* gate_up, void* out, int n, int inter, int act, int dtype,
                                          cudaStream_t stream) {
   if (n <= 0) return 0;
-  if (inter <= 0 || inter % 8 != 0 || n > 65535) return B200_ERR_BAD_SIZE;
+  if (inter <= 0 || inter % 8 != 0 || n > 65535 || (act != ACT_SILU && act != ACT_GELU_TANH)) return B200_ERR_BAD_SIZE;
   if ((reinterpret_cast<uintptr_t>(gate_up) | reinterpret_cast<uintptr_t>(out)) & 15) return B200_ERR_BAD_SIZE;
   dim3 grid((inter / 8 + 127) / 128, n);
   B200_DISPATCH_DTYPE(dtype, T,
       launch(silu_mul_interleaved_kernel<T>, grid, dim3(128), 0, stream, static_cast<const T*>(gate_up),
-             static_cast<T*>(out), inter));
+             static_cast<T*>(out), inter, act));
   return launch_status();
 }
 
@@ -792,6 +791,15 @@ __global__ void glu_limit_vec_kernel(const T* __restrict__ gate_up, T* __restric
   *reinterpret_cast<V*>(out + static_cast<size_t>(blockIdx.y) * inter + i) = Vec<T>::pack(y);
 }
 
+// x = cap * tanh(x / cap), element by element, in place (float32)
+__global__ void soft_cap_kernel(float* __restrict__ x, size_t count, float cap) {
+  pdl_trigger();
+  pdl_wait();
+  const float inv = 1.f / cap;
+  for (size_t i = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x; i < count; i += static_cast<size_t>(gridDim.x) * blockDim.x)
+    x[i] = cap * tanhf(x[i] * inv);
+}
+
 // out = relu(x)^2, element by element (float32 arithmetic, rounded once)
 template <typename T>
 __global__ void relu2_kernel(const T* __restrict__ x, T* __restrict__ out, size_t count) {
@@ -904,6 +912,16 @@ extern "C" int b200_glu_limit(const void* gate_up, void* out, int n, int inter, 
       launch(glu_limit_kernel<T>, dim3(n), dim3(256), 0, stream, static_cast<const T*>(gate_up), static_cast<T*>(out), inter, limit, alpha);
     }
   });
+  return launch_status();
+}
+
+extern "C" int b200_soft_cap(float* x, long long count, float cap, cudaStream_t stream) {
+  using namespace b200;
+  if (count <= 0) return 0;
+  if (!(cap > 0.f)) return B200_ERR_BAD_SIZE;
+  const long long blocks = (count + 255) / 256;
+  launch(soft_cap_kernel, dim3(static_cast<unsigned>(blocks < 148 * 16 ? blocks : 148 * 16)), dim3(256), 0, stream, x,
+         static_cast<size_t>(count), cap);
   return launch_status();
 }
 

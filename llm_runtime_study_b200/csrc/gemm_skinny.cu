@@ -36,10 +36,11 @@ __device__ __forceinline__ uint4 ldg_stream(const void* p) {
   return v;
 }
 
-enum Epilogue : int { EPI_STORE = 0, EPI_SWIGLU = 1, EPI_RESIDUAL = 2 };
+enum Epilogue : int { EPI_STORE = 0, EPI_SWIGLU = 1, EPI_RESIDUAL = 2 };   // EPI_SWIGLU: a gated unit, its gate by `act`
 
 // What the two fusions need beyond the product itself.
 struct NormFusion {
+  int act;                    // EPI_SWIGLU: ACT_SILU or ACT_GELU_TANH
   const float* row_scale;     // SCALED: [16] factors the rows being multiplied still lack
   const float* next_weight;   // EPI_RESIDUAL: weight of the norm that follows, [N]
   float eps;                  // EPI_RESIDUAL: its eps
@@ -160,7 +161,7 @@ gemm_skinny_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* __r
         gate += bias[n];
         up += bias[n + 8];
       }
-      C[static_cast<size_t>(m) * ldc + (n0 >> 1) + f] = from_float<OutT>(gate / (1.f + expf(-gate)) * up);
+      C[static_cast<size_t>(m) * ldc + (n0 >> 1) + f] = from_float<OutT>(gate_act(gate, fuse.act) * up);
     }
   } else {
     for (int idx = threadIdx.x; idx < 16 * NT * 8; idx += kSkinnyWarps * 32) {
@@ -265,13 +266,15 @@ static int skinny(const void* X, const void* W, const float* bias, void* C, int 
 // M <= 16, K a multiple of 8, W and X 16-byte aligned; otherwise refused.
 // `variant` picks the shape of a CTA (0: the default for the size; 2: fewer loads in flight, more CTAs per SM).
 // `swiglu` = 1: W holds gate and up rows interleaved in blocks of eight (N a multiple of 16);
-// the output is silu(gate) * up, N / 2 columns wide (ldc >= N / 2).
+// the output is silu(gate) * up, N / 2 columns wide (ldc >= N / 2); 2: gelu_tanh(gate) * up.
 // `row_scale` (optional, 16 floats): X holds rows that still lack these factors (an RMS norm left half
 // done); they are applied to the product, before the bias.
 extern "C" int b200_gemm_skinny_variant(const void* X, const void* W, const float* bias, void* C, int M, int N, int K,
                                         int ldc, int out_f32, int variant, int swiglu, const float* row_scale,
                                         cudaStream_t stream) {
+  if (swiglu < 0 || swiglu > ACT_GELU_TANH) return B200_ERR_BAD_SIZE;
   NormFusion fuse{};
+  fuse.act = swiglu;
   fuse.row_scale = row_scale;
   return skinny(X, W, bias, C, M, N, K, ldc, out_f32, variant, swiglu ? EPI_SWIGLU : EPI_STORE, fuse, stream);
 }

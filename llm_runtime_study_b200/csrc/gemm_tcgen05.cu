@@ -109,10 +109,11 @@ struct GemmParams {
   const int* tile_group;
   int group_rows;
   int act;            // 1: the square of relu on the way out (not with SWIGLU)
+  int gate_act;       // SWIGLU: ACT_SILU or ACT_GELU_TANH
 };
 
 // What the epilogue does with 32 consecutive accumulator columns of one row, starting at column nb of
-// the product: bias, then either SiLU(gate) * up on interleaved blocks of eight, or the optional sum
+// the product: bias, then either SiLU(gate) * up (or another gate) on interleaved blocks of eight, or the optional sum
 // with what C holds, then conversion and 16-byte stores where the row allows them.
 template <bool SWIGLU, typename OutT>
 __device__ __forceinline__ void finish_chunk(float (&v)[32], const GemmParams& p, OutT* crow, int nb) {
@@ -135,7 +136,7 @@ __device__ __forceinline__ void finish_chunk(float (&v)[32], const GemmParams& p
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
         const float gate = v[b * 16 + j], up = v[b * 16 + 8 + j];
-        h[b * 8 + j] = __fdividef(gate, 1.f + __expf(-gate)) * up;     // 2 ulp; for huge negative gates 0, as the limit is
+        h[b * 8 + j] = __fdividef(gate, 1.f + __expf(-gate_exponent(gate, p.gate_act))) * up;     // 2 ulp; for huge negative gates 0, as the limit is
       }
 #pragma unroll
     for (int b = 0; b < 2; ++b) {
@@ -1141,7 +1142,7 @@ extern "C" int b200_gemm_tcgen05_error() {
 // C[M,N] (ldc) = A[M,K] * W[N,K]^T + bias; out_f32 selects float or bfloat16 output.
 // K must be a multiple of 8 and both bases 16-byte aligned (TMA); refused otherwise.
 //   swiglu      W holds gate and up rows interleaved in blocks of eight (N a multiple of 16);
-//               C = silu(gate) * up with N / 2 columns (ldc >= N / 2)
+//               C = silu(gate) * up with N / 2 columns (ldc >= N / 2); 2: gelu_tanh(gate) * up
 //   accumulate  float output without swiglu: C += A W^T + bias (the residual sum done where the product is)
 //   kind        0: one CTA per 128 x tile_n tile, persistent; 1: pairs of CTAs on 256 x 256 tiles
 //               (cta_group::2); 2: stream-K (left-over tiles shared between CTAs); 3: split-K (every
@@ -1188,13 +1189,14 @@ extern "C" int b200_gemm_tcgen05(const void* A, const void* W, const float* bias
                                  int out_f32, int swiglu, int accumulate, int kind, int tile_n, int splits, int stages,
                                  float* partials, unsigned* flags, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
-  if (K <= 0 || K % 8 != 0 || ldc < (swiglu ? N / 2 : N) || (swiglu && N % 16 != 0) || kind < 0 || kind > 3) return B200_ERR_BAD_SIZE;
+  if (K <= 0 || K % 8 != 0 || ldc < (swiglu ? N / 2 : N) || (swiglu && N % 16 != 0) || swiglu < 0 || swiglu > ACT_GELU_TANH || kind < 0 || kind > 3) return B200_ERR_BAD_SIZE;
   if (kind == 1) tile_n = 256;
   if (kind != 3 && tile_n != 128 && tile_n != 256) return B200_ERR_BAD_SIZE;
   if (accumulate && (!out_f32 || swiglu)) return B200_ERR_BAD_SIZE;
   if ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(W)) & 15) return B200_ERR_BAD_SIZE;
   if (kind == 2 && (!partials || !flags || (reinterpret_cast<uintptr_t>(partials) & 15))) return 10004;
   GemmParams p{C, bias, M, N, K, ldc, (ldc % 8 == 0 && (reinterpret_cast<uintptr_t>(C) & 15) == 0) ? 1 : 0, accumulate, partials, flags, splits, BM, tile_n, 0};
+  p.gate_act = swiglu;
   CUtensorMap rows, cols;
   if (int e = make_map(&rows, A, M, K, BM)) return e;
   if (kind != 3)

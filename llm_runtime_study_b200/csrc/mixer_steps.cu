@@ -65,16 +65,38 @@ head_norm_write_kernel(const T* __restrict__ rows, int ld, T* __restrict__ q_out
   }
 }
 
+// ------------------------------------------------------------- rotation
+// Pair i of the rotated columns is (i, i + half) or, interleaved, (2i, 2i + 1): (u, v) -> (u c - v s, v c + u s) with
+// c = factor * cos(a), s = factor * sin(a), a = p * inv_freq[i].
+struct Rotation {
+  const float* inv_freq;
+  int dims;            // rotated columns, an even number
+  int interleaved;
+  float factor;
+};
+
+template <typename T>
+__device__ __forceinline__ void rotate_pair(const T* __restrict__ src, T* __restrict__ dst, int i, float p, const Rotation& rot) {
+  float sn, cs;
+  sincosf(p * rot.inv_freq[i], &sn, &cs);
+  sn *= rot.factor;
+  cs *= rot.factor;
+  const int a = rot.interleaved ? 2 * i : i, b = rot.interleaved ? 2 * i + 1 : i + rot.dims / 2;
+  const float u = to_float(src[a]), v = to_float(src[b]);
+  dst[a] = from_float<T>(u * cs - v * sn);
+  dst[b] = from_float<T>(v * cs + u * sn);
+}
+
 // ------------------------------------------------------------- latent attention: what is kept per token
 // From one stacked projection row: the query latent cols [q_off, q_off + q_rank) RMS-normed with q_w -> cq_out
 // [n, q_rank]; and, when kv_rank > 0, cols [kv_off, kv_off + kv_rank) RMS-normed with kv_w followed by `rot`
-// columns of which the first rot_dims are rotated (column i pairs with i + rot_dims/2, angle p * inv_freq[i]) ->
+// columns of which the first rot_dims are rotated (pair i turned by the angle p * inv_freq[i], see rotate_pair) ->
 // the page row [kv_rank + rot] of the token's position.
 template <typename T>
 __global__ void __launch_bounds__(256)
 latent_prepare_kernel(const T* __restrict__ rows, int ld, int q_off, int q_rank, const float* __restrict__ q_w,
-                      T* __restrict__ cq_out, int kv_off, int kv_rank, const float* __restrict__ kv_w, int rot, int rot_dims,
-                      const float* __restrict__ inv_freq, float eps, const int* __restrict__ positions,
+                      T* __restrict__ cq_out, int kv_off, int kv_rank, const float* __restrict__ kv_w, int rot,
+                      const Rotation rotation, float eps, const int* __restrict__ positions,
                       const int* __restrict__ token_entry, const int* __restrict__ block_table, int table_stride,
                       int page_size, T* __restrict__ pool) {
   __shared__ float scratch[32];
@@ -104,16 +126,9 @@ latent_prepare_kernel(const T* __restrict__ rows, int ld, int q_off, int q_rank,
   if (page < 0) return;
   T* dst = pool + (static_cast<size_t>(page) * page_size + p % page_size) * (kv_rank + rot);
   for (int i = threadIdx.x; i < kv_rank; i += blockDim.x) dst[i] = from_float<T>(to_float(row[kv_off + i]) * f * kv_w[i]);
-  const int half = rot_dims / 2;
   const T* src = row + kv_off + kv_rank;
-  for (int i = threadIdx.x; i < half; i += blockDim.x) {
-    float sn, cs;
-    sincosf(static_cast<float>(p) * inv_freq[i], &sn, &cs);
-    const float u = to_float(src[i]), v = to_float(src[i + half]);
-    dst[kv_rank + i] = from_float<T>(u * cs - v * sn);
-    dst[kv_rank + i + half] = from_float<T>(v * cs + u * sn);
-  }
-  for (int i = rot_dims + threadIdx.x; i < rot; i += blockDim.x) dst[kv_rank + i] = src[i];
+  for (int i = threadIdx.x; i < rotation.dims / 2; i += blockDim.x) rotate_pair(src, dst + kv_rank, i, static_cast<float>(p), rotation);
+  for (int i = rotation.dims + threadIdx.x; i < rot; i += blockDim.x) dst[kv_rank + i] = src[i];
 }
 
 // ------------------------------------------------------------- rotation of a slice of every head
@@ -122,25 +137,20 @@ latent_prepare_kernel(const T* __restrict__ rows, int ld, int q_off, int q_rank,
 template <typename T>
 __global__ void __launch_bounds__(128)
 rope_slice_kernel(const T* __restrict__ src, int src_ld, int src_head, int src_off, T* __restrict__ dst, int dst_ld, int dst_head,
-                  int dst_off, int heads, int rot, int rot_dims, const float* __restrict__ inv_freq,
-                  const int* __restrict__ positions) {
+                  int dst_off, int heads, int rot, const Rotation rotation, const int* __restrict__ positions) {
   pdl_trigger();
   pdl_wait();
   const int token = blockIdx.x;
   const float p = static_cast<float>(positions[token]);
-  const int half = rot_dims / 2, per_head = half + (rot - rot_dims);
+  const int half = rotation.dims / 2, per_head = half + (rot - rotation.dims);
   for (int j = threadIdx.x; j < heads * per_head; j += blockDim.x) {
     const int h = j / per_head, i = j % per_head;
     const T* s = src + static_cast<size_t>(token) * src_ld + h * src_head + src_off;
     T* o = dst + static_cast<size_t>(token) * dst_ld + h * dst_head + dst_off;
     if (i < half) {
-      float sn, cs;
-      sincosf(p * inv_freq[i], &sn, &cs);
-      const float u = to_float(s[i]), v = to_float(s[i + half]);
-      o[i] = from_float<T>(u * cs - v * sn);
-      o[i + half] = from_float<T>(v * cs + u * sn);
+      rotate_pair(s, o, i, p, rotation);
     } else {
-      o[rot_dims + i - half] = s[rot_dims + i - half];
+      o[rotation.dims + i - half] = s[rotation.dims + i - half];
     }
   }
 }
@@ -162,14 +172,14 @@ sigmoid_gate_kernel(const T* __restrict__ x, const T* __restrict__ gate, int gat
 }
 
 // ------------------------------------------------------------- norm on a sublayer's output
-// resid[t] += x[t] * rsqrt(mean(x[t]^2) + eps) * w  (x null: nothing is added); `rounded` (optional) receives the updated
+// resid[t] += factor * x[t] * rsqrt(mean(x[t]^2) + eps) * w  (x null: nothing is added); `rounded` (optional) receives the updated
 // rows in the activation type, for the sublayer that reads them next.  The sublayer's output row may be given in pieces:
 // with pair_row, row t of x is sum_j pair_w[t, j] * x[pair_row[t, j]] (j ascending; what a router's experts returned for the
 // token), formed here instead of by a launch of its own.  The row is kept in shared memory between the two passes.
 template <typename T>
 __global__ void __launch_bounds__(256)
 norm_accumulate_round_kernel(const float* __restrict__ x, const float* __restrict__ w, float* __restrict__ resid,
-                             T* __restrict__ rounded, int hidden, float eps, const int* __restrict__ pair_row,
+                             T* __restrict__ rounded, int hidden, float eps, float factor, const int* __restrict__ pair_row,
                              const float* __restrict__ pair_w, int top) {
   __shared__ float scratch[32];
   extern __shared__ __align__(16) float kept[];
@@ -201,7 +211,7 @@ norm_accumulate_round_kernel(const float* __restrict__ x, const float* __restric
         ss = fmaf(kept[i], kept[i], ss);
       }
     }
-    f = rsqrtf(block_sum(ss, scratch) / static_cast<float>(hidden) + eps);
+    f = rsqrtf(block_sum(ss, scratch) / static_cast<float>(hidden) + eps) * factor;
   }
   if ((hidden & 3) == 0 && x != nullptr) {
     for (int i = threadIdx.x; i < hidden / 4; i += blockDim.x) {
@@ -256,7 +266,8 @@ extern "C" int b200_head_norm_write(const void* rows, int ld, void* q_out, const
 }
 
 extern "C" int b200_latent_prepare(const void* rows, int ld, int q_off, int q_rank, const float* q_w, void* cq_out, int kv_off,
-                                   int kv_rank, const float* kv_w, int rot, int rot_dims, const float* inv_freq, float eps,
+                                   int kv_rank, const float* kv_w, int rot, int rot_dims, const float* inv_freq, int interleaved,
+                                   float rot_factor, float eps,
                                    const int* positions, const int* token_entry, const int* block_table, int table_stride,
                                    int page_size, void* pool, int n, int dtype, cudaStream_t stream) {
   using namespace b200;
@@ -265,21 +276,22 @@ extern "C" int b200_latent_prepare(const void* rows, int ld, int q_off, int q_ra
       (kv_rank > 0 && (kv_off < 0 || kv_off + kv_rank + rot > ld || page_size <= 0)))
     return B200_ERR_BAD_SIZE;
   B200_DISPATCH_DTYPE(dtype, T, launch(latent_prepare_kernel<T>, dim3(n), dim3(256), 0, stream, static_cast<const T*>(rows), ld, q_off,
-                                       q_rank, q_w, static_cast<T*>(cq_out), kv_off, kv_rank, kv_w, rot, rot_dims, inv_freq, eps,
+                                       q_rank, q_w, static_cast<T*>(cq_out), kv_off, kv_rank, kv_w, rot,
+                                       Rotation{inv_freq, rot_dims, interleaved, rot_factor}, eps,
                                        positions, token_entry, block_table, table_stride, page_size, static_cast<T*>(pool)));
   return launch_status();
 }
 
 extern "C" int b200_rope_slice(const void* src, int src_ld, int src_head, int src_off, void* dst, int dst_ld, int dst_head,
-                               int dst_off, int heads, int rot, int rot_dims, const float* inv_freq, const int* positions, int n,
-                               int dtype, cudaStream_t stream) {
+                               int dst_off, int heads, int rot, int rot_dims, const float* inv_freq, int interleaved, float rot_factor,
+                               const int* positions, int n, int dtype, cudaStream_t stream) {
   using namespace b200;
   if (n <= 0 || rot <= 0) return 0;
   if (heads <= 0 || rot_dims < 0 || rot_dims > rot || rot_dims % 2 || src_off + rot > src_head || dst_off + rot > dst_head)
     return B200_ERR_BAD_SIZE;
   B200_DISPATCH_DTYPE(dtype, T, launch(rope_slice_kernel<T>, dim3(n), dim3(128), 0, stream, static_cast<const T*>(src), src_ld,
-                                       src_head, src_off, static_cast<T*>(dst), dst_ld, dst_head, dst_off, heads, rot, rot_dims,
-                                       inv_freq, positions));
+                                       src_head, src_off, static_cast<T*>(dst), dst_ld, dst_head, dst_off, heads, rot,
+                                       Rotation{inv_freq, rot_dims, interleaved, rot_factor}, positions));
   return launch_status();
 }
 
@@ -294,13 +306,13 @@ extern "C" int b200_sigmoid_gate(const void* x, const void* gate, int gate_ld, i
 }
 
 extern "C" int b200_norm_accumulate_round(const float* x, const float* w, float* resid, void* rounded, int n, int hidden, float eps,
-                                          const int* pair_row, const float* pair_w, int top, int dtype, cudaStream_t stream) {
+                                          float factor, const int* pair_row, const float* pair_w, int top, int dtype, cudaStream_t stream) {
   using namespace b200;
   if (n <= 0) return 0;
   if (hidden <= 0 || hidden > 12288 || (pair_row != nullptr && (pair_w == nullptr || top <= 0 || x == nullptr))) return B200_ERR_BAD_SIZE;
   if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(resid)) & 15) return B200_ERR_BAD_SIZE;
   const size_t smem = x != nullptr ? sizeof(float) * hidden : 0;
   B200_DISPATCH_DTYPE(dtype, T, launch(norm_accumulate_round_kernel<T>, dim3(n), dim3(256), smem, stream, x, w, resid,
-                                       static_cast<T*>(rounded), hidden, eps, pair_row, pair_w, top));
+                                       static_cast<T*>(rounded), hidden, eps, factor, pair_row, pair_w, top));
   return launch_status();
 }

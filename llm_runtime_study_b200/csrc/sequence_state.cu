@@ -2,10 +2,14 @@
 //
 //   linear scan     S_t = D_t S_(t-1) + k_t u_t^T,  o_t = S_t^T q_t        per head, S is [d, dv]
 //                   (the delta rule's read-out is formed as (D_t S_(t-1))^T q_t + u_t (k_t . q_t), the same sum)
-//                   D_t = one decay per head (a constant), or a diagonal of per-row factors g_t (gated)
-//                   u_t = v_t (plain), or beta_t (v_t - (D_t S_(t-1))^T k_t) (delta rule)
+//                   D_t = one decay per head (a constant), a diagonal of per-row factors g_t (gated), or one factor per
+//                         row and head (row gates)
+//                   u_t = v_t (plain), beta_t (v_t - (D_t S_(t-1))^T k_t) (delta rule), or b_t v_t (row gates, which also
+//                         carry n_t = D_t n_(t-1) + b_t k_t and give n_t . q_t: the matrix memory's normaliser)
 //   short convolution over time per channel, with the last taps-1 inputs kept per request
-//   per-group RMS norm of the read-out times a sigmoid gate
+//   per-group RMS norm of the read-out times a sigmoid or SiLU gate
+//   the gates themselves: exponential input and forget gates kept in range by a running maximum, decays per key channel
+//                   from a low-rank map
 //
 // The state, the decays, the gates of the recurrence and the unit norms are float32 whatever the
 // storage type of the projections.  Tokens of one request are processed in order, one after the
@@ -18,6 +22,8 @@ namespace b200 {
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float silu_f(float x) { return x * sigmoid_f(x); }
 __device__ __forceinline__ float softplus_f(float x) { return x > 20.f ? x : log1pf(expf(x)); }
+// ln sigmoid(x), without a cancellation on either side of zero
+__device__ __forceinline__ float log_sigmoid_f(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
 // SiLU of a value that was stored in 16 bits: the hardware's exponential and reciprocal are exact far beyond the
 // 8 bits of such a value; 32-bit inputs take the full-precision functions.
 template <typename T> __device__ __forceinline__ float silu_of(float x) {
@@ -36,7 +42,12 @@ struct ScanParams {
   float* out; int ldo;                            // [n, H * dv]
   const int* q_start; const int* slots;           // per entry: first token, request slot
   int H, Hqk, d, dv, act, rl;                     // act 1: silu on q, k, v as they are read; rl: lanes that share a column
+  const float* row_decay; const float* row_gain;  // [n, H]: D_t and b_t (row gates)
+  float* norm_state; float* norm_out;             // [slots, H, d], [n, H]: n and n . q (row gates)
+  float q_scale;                                  // on q as it is read
 };
+
+enum ScanGate : int { GATE_HEAD = 0, GATE_CHANNEL = 1, GATE_ROW = 2 };
 
 constexpr int kScanThreads = 128;
 // tokens staged in shared memory at a time: 16, or 8 where a token's rows are more than 128 wide
@@ -51,36 +62,45 @@ constexpr int scan_chunk(int dpt, int rl) { return dpt * rl <= 128 ? 16 : 8; }
 // RL = 16 spreads a column over more lanes and a head over sixteen times as many CTAs, which is
 // what a launch with few requests and long portions wants: its time is a chain of dependent steps,
 // and the chain per token is a quarter as long.
-template <typename T, int DPT, int RL, bool DELTA, bool GATED>
+// GATE_ROW: the normaliser n is one more column of the state, behind the last value column, whose value is 1 for every
+// token; it lives in an array of its own.
+template <typename T, int DPT, int RL, bool DELTA, int GATE>
 __global__ void __launch_bounds__(kScanThreads) linear_scan_kernel(const ScanParams p) {
   extern __shared__ __align__(16) float smem[];
   pdl_trigger();
   pdl_wait();
+  constexpr bool GATED = GATE == GATE_CHANNEL, ROW = GATE == GATE_ROW;
+  static_assert(!(DELTA && ROW), "row gates and the delta rule exclude each other");
   constexpr int rl = RL, cols_per_warp = 32 / rl, cols = (kScanThreads / 32) * cols_per_warp;
   constexpr int dp = DPT * rl;                          // rows padded to dp >= d; the padding holds zeros
   constexpr int CHUNK = scan_chunk(DPT, RL);            // tokens staged in shared memory at a time
   constexpr int EPT = CHUNK * dp / kScanThreads;        // staged elements of k (q, g) per thread
   constexpr int VPT = (CHUNK * cols + kScanThreads - 1) / kScanThreads;
-  const int col_blocks = (p.dv + cols - 1) / cols;
+  const int col_blocks = (p.dv + (ROW ? 1 : 0) + cols - 1) / cols;
   const int h = blockIdx.x / col_blocks, cb = blockIdx.x % col_blocks;
   const int entry = blockIdx.y;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int r = lane / cols_per_warp;
   const int col_local = warp * cols_per_warp + lane % cols_per_warp;
   const int col = cb * cols + col_local;
-  const bool live = col < p.dv;
   const int d = p.d, dv = p.dv;
+  const bool is_norm = ROW && col == dv;
+  const bool live = col < dv || is_norm;
   const int hqk = h / (p.H / p.Hqk);
   const int t_begin = p.q_start[entry], t_end = p.q_start[entry + 1];
   const int slot = p.slots[entry];
-  float* sbase = p.state + (static_cast<size_t>(slot) * p.H + h) * d * dv;
+  // this column's entries: sbase[i * srow]
+  float* sbase = is_norm ? p.norm_state + (static_cast<size_t>(slot) * p.H + h) * d
+                         : p.state + (static_cast<size_t>(slot) * p.H + h) * d * dv + col;
+  const int srow = is_norm ? 1 : dv;
 
   float* ks = smem;                              // [chunk][dp]
   float* qs = ks + CHUNK * dp;                   // [chunk][dp]
   float* gs = qs + CHUNK * dp;                   // [chunk][dp] (gated only)
   float* vs = gs + (GATED ? CHUNK * dp : 0);     // [chunk][cols]
-  float* bs = vs + CHUNK * cols;                 // [chunk]
-  const float dec = GATED ? 1.f : p.decay[h];
+  float* bs = vs + CHUNK * cols;                 // [chunk]: beta (delta rule) or b (row gates)
+  float* ds = bs + CHUNK;                        // [chunk]: the head's factor of the token (row gates)
+  float dec = GATE == GATE_HEAD ? p.decay[h] : 1.f;
   const T* qg = static_cast<const T*>(p.q);
   const T* kg = static_cast<const T*>(p.k);
   const T* vg = static_cast<const T*>(p.v);
@@ -89,7 +109,7 @@ __global__ void __launch_bounds__(kScanThreads) linear_scan_kernel(const ScanPar
   // registers; they go to shared memory (SiLU applied once per element) when this chunk is done.
   // (kept in the storage type: a conversion right behind the load would wait for it)
   T rk[EPT], rq[EPT], rv[VPT];
-  float rg[EPT], rb = 0.f;
+  float rg[EPT], rb = 0.f, rd = 0.f;
   auto fetch = [&](int t0, int count) {
 #pragma unroll
     for (int e = 0; e < EPT; ++e) {
@@ -110,9 +130,13 @@ __global__ void __launch_bounds__(kScanThreads) linear_scan_kernel(const ScanPar
       if (e * kScanThreads >= count * cols) break;
       const int idx = threadIdx.x + e * kScanThreads;
       const int tt = idx / cols, c = cb * cols + idx % cols;
-      rv[e] = (tt < count && c < dv) ? vg[static_cast<size_t>(t0 + tt) * p.ldv + h * dv + c] : from_float<T>(0.f);
+      rv[e] = (tt < count && c < dv) ? vg[static_cast<size_t>(t0 + tt) * p.ldv + h * dv + c] : from_float<T>(ROW && c == dv ? 1.f : 0.f);
     }
     if (DELTA && threadIdx.x < count) rb = p.beta[static_cast<size_t>(t0 + threadIdx.x) * p.ldb + h];
+    if (ROW && threadIdx.x < count) {
+      rb = p.row_gain[static_cast<size_t>(t0 + threadIdx.x) * p.H + h];
+      rd = p.row_decay[static_cast<size_t>(t0 + threadIdx.x) * p.H + h];
+    }
   };
   auto stash = [&](int count) {
 #pragma unroll
@@ -120,7 +144,7 @@ __global__ void __launch_bounds__(kScanThreads) linear_scan_kernel(const ScanPar
       if (e * kScanThreads >= count * dp) break;
       const int idx = threadIdx.x + e * kScanThreads;
       ks[idx] = p.act ? silu_of<T>(to_float(rk[e])) : to_float(rk[e]);
-      qs[idx] = p.act ? silu_of<T>(to_float(rq[e])) : to_float(rq[e]);
+      qs[idx] = (p.act ? silu_of<T>(to_float(rq[e])) : to_float(rq[e])) * p.q_scale;
       if (GATED) gs[idx] = rg[e];
     }
 #pragma unroll
@@ -129,7 +153,8 @@ __global__ void __launch_bounds__(kScanThreads) linear_scan_kernel(const ScanPar
       const int idx = threadIdx.x + e * kScanThreads;
       if (idx < CHUNK * cols) vs[idx] = p.act ? silu_of<T>(to_float(rv[e])) : to_float(rv[e]);
     }
-    if (DELTA && threadIdx.x < CHUNK) bs[threadIdx.x] = rb;
+    if ((DELTA || ROW) && threadIdx.x < CHUNK) bs[threadIdx.x] = rb;
+    if (ROW && threadIdx.x < CHUNK) ds[threadIdx.x] = rd;
   };
 
   fetch(t_begin, min(CHUNK, t_end - t_begin));
@@ -137,7 +162,7 @@ __global__ void __launch_bounds__(kScanThreads) linear_scan_kernel(const ScanPar
 #pragma unroll
   for (int ii = 0; ii < DPT; ++ii) {
     const int i = r * DPT + ii;
-    S[ii] = (live && i < d) ? sbase[static_cast<size_t>(i) * dv + col] : 0.f;
+    S[ii] = (live && i < d) ? sbase[static_cast<size_t>(i) * srow] : 0.f;
   }
 
   for (int t0 = t_begin; t0 < t_end; t0 += CHUNK) {
@@ -196,7 +221,8 @@ __global__ void __launch_bounds__(kScanThreads) linear_scan_kernel(const ScanPar
           S[4 * v + 3] = fmaf(kk[v].w, u, S[4 * v + 3]);
         }
       } else {
-        const float u = vs[tt * cols + col_local];
+        const float u = ROW ? vs[tt * cols + col_local] * bs[tt] : vs[tt * cols + col_local];
+        if (ROW) dec = ds[tt];
         float acc[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
         for (int v = 0; v < DPT / 4; ++v) {
@@ -221,29 +247,34 @@ __global__ void __launch_bounds__(kScanThreads) linear_scan_kernel(const ScanPar
 #pragma unroll
         for (int o = cols_per_warp; o < 32; o <<= 1) o_sum += __shfl_xor_sync(0xffffffffu, o_sum, o);
       }
-      if (live && r == 0) p.out[static_cast<size_t>(t0 + tt) * p.ldo + h * dv + col] = o_sum;
+      if (live && r == 0) {
+        if (is_norm) p.norm_out[static_cast<size_t>(t0 + tt) * p.H + h] = o_sum;
+        else p.out[static_cast<size_t>(t0 + tt) * p.ldo + h * dv + col] = o_sum;
+      }
     }
   }
 #pragma unroll
   for (int ii = 0; ii < DPT; ++ii) {
     const int i = r * DPT + ii;
-    if (live && i < d) sbase[static_cast<size_t>(i) * dv + col] = S[ii];
+    if (live && i < d) sbase[static_cast<size_t>(i) * srow] = S[ii];
   }
 }
 
-template <typename T, bool DELTA, bool GATED>
+template <typename T, bool DELTA, int GATE>
 int launch_scan(ScanParams p, int entries, cudaStream_t stream) {
   const int dpt = (p.d + p.rl - 1) / p.rl;
   const int cols = (kScanThreads / 32) * (32 / p.rl);
-  dim3 grid(p.H * ((p.dv + cols - 1) / cols), entries);
+  constexpr bool GATED = GATE == GATE_CHANNEL;
+  const int columns = p.dv + (GATE == GATE_ROW ? 1 : 0);
+  dim3 grid(p.H * ((columns + cols - 1) / cols), entries);
   if (grid.y > 65535) return B200_ERR_TOO_LARGE;
   const int dpt8 = (dpt + 7) / 8 * 8;
   const int chunk = scan_chunk(dpt8, p.rl);
-  const size_t smem = sizeof(float) * (static_cast<size_t>(chunk) * dpt8 * p.rl * (GATED ? 3 : 2) + chunk * cols + chunk);
+  const size_t smem = sizeof(float) * (static_cast<size_t>(chunk) * dpt8 * p.rl * (GATED ? 3 : 2) + chunk * cols + 2 * chunk);
   if (smem > 48 * 1024) return B200_ERR_TOO_LARGE;
 #define B200_SCAN_CASE(DPT_, RL_)                                                                                      \
   if (dpt8 == DPT_ && p.rl == RL_) {                                                                                   \
-    launch(linear_scan_kernel<T, DPT_, RL_, DELTA, GATED>, grid, dim3(kScanThreads), smem, stream, p);                 \
+    launch(linear_scan_kernel<T, DPT_, RL_, DELTA, GATE>, grid, dim3(kScanThreads), smem, stream, p);                 \
     return launch_status();                                                                                            \
   }
   B200_SCAN_CASE(8, 4) B200_SCAN_CASE(16, 4) B200_SCAN_CASE(24, 4) B200_SCAN_CASE(32, 4)
@@ -360,6 +391,89 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const DeltaPreparePa
   }
 }
 
+// ------------------------------------------------------------- exponential gates of a matrix memory
+// Per request and head, token after token: with i = cap tanh((zi + bi) / cap) and f = ln sigmoid(cap tanh((zf + bf) / cap)),
+//   m_t = max(f + m_(t-1), i),  decay = exp(f + m_(t-1) - m_t),  gain = exp(i - m_t),  floor = exp(-m_t)
+// from the slot's m (0 for a new request).  One warp per head: the lanes form i and f of 32 tokens, every lane walks the
+// chain of maxima (an addition and a maximum a token), the lanes form the exponentials.
+constexpr int kGateWarps = 4;
+template <typename T>
+__global__ void __launch_bounds__(kGateWarps * 32)
+memory_gates_kernel(const T* __restrict__ proj, int ld, int i_off, int f_off, const float* __restrict__ i_bias,
+                    const float* __restrict__ f_bias, float cap, float* __restrict__ m_state, float* __restrict__ decay,
+                    float* __restrict__ gain, float* __restrict__ floor_, const int* __restrict__ q_start,
+                    const int* __restrict__ slots, int H) {
+  pdl_trigger();
+  pdl_wait();
+  const int lane = threadIdx.x & 31, h = blockIdx.x * kGateWarps + (threadIdx.x >> 5), entry = blockIdx.y;
+  if (h >= H) return;
+  const int t_end = q_start[entry + 1], t_begin = q_start[entry];
+  float* kept = m_state + static_cast<size_t>(slots[entry]) * H + h;
+  const float bi = i_bias[h], bf = f_bias[h];
+  float m = *kept;
+  float zi = 0.f, zf = 0.f;
+  auto fetch = [&](int t) {
+    if (t < t_end) {
+      zi = to_float(proj[static_cast<size_t>(t) * ld + i_off + h]);
+      zf = to_float(proj[static_cast<size_t>(t) * ld + f_off + h]);
+    }
+  };
+  fetch(t_begin + lane);
+  for (int t0 = t_begin; t0 < t_end; t0 += 32) {
+    const float li = cap * tanhf((zi + bi) / cap), lf = log_sigmoid_f(cap * tanhf((zf + bf) / cap));
+    fetch(t0 + 32 + lane);
+    const int count = min(32, t_end - t0);
+    float before = 0.f, after = 0.f;
+    for (int j = 0; j < count; ++j) {
+      const float fj = __shfl_sync(0xffffffffu, lf, j), ij = __shfl_sync(0xffffffffu, li, j);
+      const float m_new = fmaxf(fj + m, ij);
+      if (lane == j) {
+        before = m;
+        after = m_new;
+      }
+      m = m_new;
+    }
+    if (lane < count) {
+      const size_t at = static_cast<size_t>(t0 + lane) * H + h;
+      decay[at] = expf(lf + before - after);
+      gain[at] = expf(li - after);
+      floor_[at] = expf(-after);
+    }
+  }
+  if (lane == 0) *kept = m;
+}
+
+// ------------------------------------------------------------- decays per key channel
+// alpha[t, c] = sigmoid(sum_j up[j, c] * proj[t, off + j] + bias[c])^(1 / tau): a thread owns a column for TOKENS tokens, so
+// that its column of the low-rank map is fetched once for all of them; up is [rank, width], the map's weight transposed.
+template <typename T, int TOKENS>
+__global__ void __launch_bounds__(128)
+channel_decay_kernel(const T* __restrict__ proj, int ld, int off, int rank, const T* __restrict__ up, const float* __restrict__ bias,
+                     float inv_tau, float* __restrict__ alpha, int n, int width) {
+  extern __shared__ float low[];       // [TOKENS][rank]
+  pdl_trigger();
+  pdl_wait();
+  const int t0 = blockIdx.x * TOKENS, count = min(TOKENS, n - t0);
+  for (int idx = threadIdx.x; idx < count * rank; idx += blockDim.x)
+    low[idx] = to_float(proj[static_cast<size_t>(t0 + idx / rank) * ld + off + idx % rank]);
+  __syncthreads();
+  const int c = blockIdx.y * blockDim.x + threadIdx.x;
+  if (c >= width) return;
+  float z[TOKENS];
+#pragma unroll
+  for (int k = 0; k < TOKENS; ++k) z[k] = 0.f;
+  for (int j = 0; j < rank; ++j) {
+    const float u = to_float(up[static_cast<size_t>(j) * width + c]);
+#pragma unroll
+    for (int k = 0; k < TOKENS; ++k)
+      if (k < count) z[k] = fmaf(u, low[k * rank + j], z[k]);
+  }
+  const float b = bias[c];
+#pragma unroll
+  for (int k = 0; k < TOKENS; ++k)
+    if (k < count) alpha[static_cast<size_t>(t0 + k) * width + c] = expf(log_sigmoid_f(z[k] + b) * inv_tau);
+}
+
 // After a step: the last taps-1 inputs of each request, from the step's rows and, where the step
 // was shorter than that, from what the state held.  One thread per channel walks the rows oldest
 // first; row s is written after row len + s (> s) has been read, so nothing is read after it changed.
@@ -381,13 +495,15 @@ __global__ void conv_state_update_kernel(const T* __restrict__ proj, int ld, flo
 }
 
 // ------------------------------------------------------------- group norm times sigmoid gate
-// out[t, c] = x[t, c] * rsqrt(mean over c's group of x^2 + eps) * w[c % group] * sigmoid(gate[t, c]);
-// the gate's logits are read from `gate_in` directly (rank 0) or formed as gate_up[:, c] . gate_in[t, :rank]
+// out[t, c] = y[t, c] * rsqrt(mean over c's group of y^2 + eps) * w[c % w_len] * act(gate[t, c]), act the sigmoid or SiLU;
+// y = x, or, with `den` and `floor` ([n, width / group] each), y = x / (max(|den|, floor) + den_eps) with its group's two
+// numbers.  w_len is the group's size (one weight for all groups) or the width.  The gate's logits are read from `gate_in` directly (rank 0) or formed as gate_up[:, c] . gate_in[t, :rank]
 // (gate_up is [rank, width]: the map's weight transposed).
 template <typename T>
-__global__ void group_norm_gate_kernel(const float* __restrict__ x, int width, int group, const float* __restrict__ w, float eps,
+__global__ void group_norm_gate_kernel(const float* __restrict__ x, int width, int group, const float* __restrict__ w, int w_len,
+                                       float eps, const float* __restrict__ den, const float* __restrict__ floor_, float den_eps,
                                        const T* __restrict__ gate_in, int gate_ld, int rank, const T* __restrict__ gate_up,
-                                       T* __restrict__ out) {
+                                       int gate_silu, T* __restrict__ out) {
   __shared__ float scratch[32];
   extern __shared__ float low[];
   pdl_trigger();
@@ -397,7 +513,14 @@ __global__ void group_norm_gate_kernel(const float* __restrict__ x, int width, i
   for (int j = threadIdx.x; j < rank; j += blockDim.x) low[j] = to_float(gate_in[static_cast<size_t>(t) * gate_ld + j]);
   float ss = 0.f;
   for (int i = threadIdx.x; i < group; i += blockDim.x) ss = fmaf(row[i], row[i], ss);
-  const float f = rsqrtf(block_sum(ss, scratch) / static_cast<float>(group) + eps);
+  float inv = 1.f;
+  if (den != nullptr) {
+    const size_t at = static_cast<size_t>(t) * gridDim.y + blockIdx.y;
+    inv = 1.f / (fmaxf(fabsf(den[at]), floor_[at]) + den_eps);
+  }
+  // (the mean of squares of x times inv^2, in this order: x * inv squared would not overflow any later)
+  const float f = inv * rsqrtf(block_sum(ss, scratch) / static_cast<float>(group) * inv * inv + eps);
+  const float* wg = w_len == group ? w : w + base;
   for (int i = threadIdx.x; i < group; i += blockDim.x) {
     const int c = base + i;
     float logit;
@@ -407,7 +530,7 @@ __global__ void group_norm_gate_kernel(const float* __restrict__ x, int width, i
       logit = 0.f;
       for (int j = 0; j < rank; ++j) logit = fmaf(to_float(gate_up[static_cast<size_t>(j) * width + c]), low[j], logit);
     }
-    out[static_cast<size_t>(t) * width + c] = from_float<T>(row[i] * f * w[i] * sigmoid_f(logit));
+    out[static_cast<size_t>(t) * width + c] = from_float<T>(row[i] * f * wg[i] * (gate_silu ? silu_f(logit) : sigmoid_f(logit)));
   }
 }
 
@@ -420,24 +543,71 @@ __global__ void group_norm_gate_kernel(const float* __restrict__ x, int width, i
 extern "C" int b200_linear_scan(const void* q, const void* k, const void* v, int ldq, int ldk, int ldv, const float* gate, int ldg,
                                 const float* decay, const float* beta, int ldb, float* state, float* out, int ldo,
                                 const int* q_start, const int* slots, int entries, int tokens, int H, int Hqk, int d, int dv,
-                                int act, int fixed_order, int dtype, cudaStream_t stream) {
+                                int act, float q_scale, int fixed_order, int dtype, cudaStream_t stream) {
   using namespace b200;
   if (entries <= 0) return 0;
   if (H <= 0 || Hqk <= 0 || H % Hqk != 0 || d <= 0 || dv <= 0 || d > 256) return B200_ERR_BAD_SIZE;
   if ((gate == nullptr) == (decay == nullptr)) return B200_ERR_BAD_SIZE;
-  ScanParams p{q, k, v, ldq, ldk, ldv, gate, ldg, decay, beta, ldb, state, out, ldo, q_start, slots, H, Hqk, d, dv, act, 1};
+  ScanParams p{q, k, v, ldq, ldk, ldv, gate, ldg, decay, beta, ldb, state, out, ldo, q_start, slots, H, Hqk, d, dv, act, 1, nullptr, nullptr, nullptr, nullptr, q_scale};
   p.rl = scan_row_lanes(entries, H, d, dv, tokens, fixed_order);
   const bool delta = beta != nullptr, gated = gate != nullptr;
   if (delta && gated) {
-    B200_DISPATCH_DTYPE(dtype, T, return (launch_scan<T, true, true>(p, entries, stream)));
+    B200_DISPATCH_DTYPE(dtype, T, return (launch_scan<T, true, GATE_CHANNEL>(p, entries, stream)));
   } else if (!delta && !gated) {
-    B200_DISPATCH_DTYPE(dtype, T, return (launch_scan<T, false, false>(p, entries, stream)));
+    B200_DISPATCH_DTYPE(dtype, T, return (launch_scan<T, false, GATE_HEAD>(p, entries, stream)));
   } else if (delta) {
-    B200_DISPATCH_DTYPE(dtype, T, return (launch_scan<T, true, false>(p, entries, stream)));
+    B200_DISPATCH_DTYPE(dtype, T, return (launch_scan<T, true, GATE_HEAD>(p, entries, stream)));
   } else {
-    B200_DISPATCH_DTYPE(dtype, T, return (launch_scan<T, false, true>(p, entries, stream)));
+    B200_DISPATCH_DTYPE(dtype, T, return (launch_scan<T, false, GATE_CHANNEL>(p, entries, stream)));
   }
   return 0;
+}
+
+// The scan with row gates: S <- decay[t, h] S + gain[t, h] k v^T, n <- decay[t, h] n + gain[t, h] k, out = S^T q, norm_out = n . q
+// (q times q_scale as it is read); state [slots, H, d, dv] and norm_state [slots, H, d] float32, decay, gain, norm_out [n, H].
+extern "C" int b200_linear_scan_row_gates(const void* q, const void* k, const void* v, int ldq, int ldk, int ldv, const float* decay,
+                                          const float* gain, float* state, float* norm_state, float* out, float* norm_out,
+                                          const int* q_start, const int* slots, int entries, int tokens, int H, int d, int dv,
+                                          float q_scale, int fixed_order, int dtype, cudaStream_t stream) {
+  using namespace b200;
+  if (entries <= 0) return 0;
+  if (H <= 0 || d <= 0 || dv <= 0 || d > 256 || !decay || !gain || !norm_state || !norm_out) return B200_ERR_BAD_SIZE;
+  ScanParams p{q, k, v, ldq, ldk, ldv, nullptr, 0, nullptr, nullptr, 0, state, out, H * dv, q_start, slots, H, H, d, dv, 0, 1,
+               decay, gain, norm_state, norm_out, q_scale};
+  p.rl = scan_row_lanes(entries, H, d, dv + 1, tokens, fixed_order);
+  B200_DISPATCH_DTYPE(dtype, T, return (launch_scan<T, false, GATE_ROW>(p, entries, stream)));
+  return 0;
+}
+
+extern "C" int b200_memory_gates(const void* proj, int ld, int i_off, int f_off, const float* i_bias, const float* f_bias, float cap,
+                                 float* m_state, float* decay, float* gain, float* floor_, const int* q_start, const int* slots,
+                                 int entries, int H, int dtype, cudaStream_t stream) {
+  using namespace b200;
+  if (entries <= 0) return 0;
+  if (H <= 0 || entries > 65535 || !(cap > 0.f) || i_off < 0 || f_off < 0 || i_off + H > ld || f_off + H > ld) return B200_ERR_BAD_SIZE;
+  dim3 grid((H + kGateWarps - 1) / kGateWarps, entries);
+  B200_DISPATCH_DTYPE(dtype, T, launch(memory_gates_kernel<T>, grid, dim3(kGateWarps * 32), 0, stream, static_cast<const T*>(proj), ld,
+                                       i_off, f_off, i_bias, f_bias, cap, m_state, decay, gain, floor_, q_start, slots, H));
+  return launch_status();
+}
+
+extern "C" int b200_channel_decay(const void* proj, int ld, int off, int rank, const void* up, const float* bias, float tau, float* alpha,
+                                  int n, int width, int dtype, cudaStream_t stream) {
+  using namespace b200;
+  if (n <= 0) return 0;
+  if (rank <= 0 || rank > 1024 || width <= 0 || !(tau > 0.f) || off < 0 || off + rank > ld) return B200_ERR_BAD_SIZE;
+  const int blocks = (width + 127) / 128;
+  if (blocks > 65535) return B200_ERR_TOO_LARGE;
+  if (n >= 64) {        // portions of prompts: eight tokens share a fetch of the map
+    B200_DISPATCH_DTYPE(dtype, T, launch(channel_decay_kernel<T, 8>, dim3((n + 7) / 8, blocks), dim3(128), sizeof(float) * 8 * rank, stream,
+                                         static_cast<const T*>(proj), ld, off, rank, static_cast<const T*>(up), bias, 1.f / tau, alpha, n,
+                                         width));
+  } else {
+    B200_DISPATCH_DTYPE(dtype, T, launch(channel_decay_kernel<T, 1>, dim3(n, blocks), dim3(128), sizeof(float) * rank, stream,
+                                         static_cast<const T*>(proj), ld, off, rank, static_cast<const T*>(up), bias, 1.f / tau, alpha, n,
+                                         width));
+  }
+  return launch_status();
 }
 
 extern "C" int b200_delta_prepare(const void* proj, int ld, int b_off, int a_off, int rank, const float* taps, int ntaps,
@@ -479,16 +649,19 @@ extern "C" int b200_conv_state_update(const void* proj, int ld, float* conv_stat
   return launch_status();
 }
 
-extern "C" int b200_group_norm_gate(const float* x, int n, int width, int group, const float* w, float eps, const void* gate_in,
-                                    int gate_ld, int rank, const void* gate_up, void* out, int dtype, cudaStream_t stream) {
+extern "C" int b200_group_norm_gate(const float* x, int n, int width, int group, const float* w, int w_len, float eps, const float* den,
+                                    const float* floor_, float den_eps, const void* gate_in, int gate_ld, int rank,
+                                    const void* gate_up, int gate_silu, void* out, int dtype, cudaStream_t stream) {
   using namespace b200;
   if (n <= 0) return 0;
-  if (width <= 0 || group <= 0 || width % group != 0 || rank < 0 || rank > 4096) return B200_ERR_BAD_SIZE;
+  if (width <= 0 || group <= 0 || width % group != 0 || rank < 0 || rank > 4096 || (w_len != group && w_len != width) ||
+      (den == nullptr) != (floor_ == nullptr))
+    return B200_ERR_BAD_SIZE;
   dim3 grid(n, width / group);
   if (grid.y > 65535) return B200_ERR_TOO_LARGE;
   const int threads = group >= 256 ? 256 : (group + 31) / 32 * 32;
   B200_DISPATCH_DTYPE(dtype, T, launch(group_norm_gate_kernel<T>, grid, dim3(threads), sizeof(float) * rank, stream, x, width, group,
-                                       w, eps, static_cast<const T*>(gate_in), gate_ld, rank, static_cast<const T*>(gate_up),
-                                       static_cast<T*>(out)));
+                                       w, w_len, eps, den, floor_, den_eps, static_cast<const T*>(gate_in), gate_ld, rank,
+                                       static_cast<const T*>(gate_up), gate_silu, static_cast<T*>(out)));
   return launch_status();
 }

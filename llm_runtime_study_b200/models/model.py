@@ -95,7 +95,9 @@ class DecoderModel:
             first = self.embedding.forward(ctx.token_ids, next_norm=None if 0 in steps else blocks[0].first_norm())
         else:
             first = self.embedding.forward(ctx.token_ids)
-        if isinstance(first, tuple):     # (rows, the same rows prepared for the first norm)
+        if isinstance(first, ResidualStream):
+            stream = first
+        elif isinstance(first, tuple):     # (rows, the same rows prepared for the first norm)
             stream = ResidualStream(first[0], weighted=first[1], weighted_for=blocks[0].first_norm())
         else:
             stream = ResidualStream(first)

@@ -22,7 +22,7 @@ _TABLE = {
     "b200_attention_latent_rank": [],
     "b200_attention_latent_rot": [],
     "b200_attention_latent_bf16": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int,
-                                   c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, ctypes.c_long, c_void_p],
+                                   c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, ctypes.c_long, c_void_p],
 }
 
 
@@ -48,9 +48,10 @@ def build(rank: int, rot: int) -> None:
 
 
 def latent_attention(q: torch.Tensor, pool: torch.Tensor, ctx: Any, table: torch.Tensor, *, value_dim: int, scale: float,
-                     window: int = 0) -> torch.Tensor:
+                     window: int = 0, sink: torch.Tensor | None = None) -> torch.Tensor:
     """Causal attention of the batch's query tokens ``[N, heads, d]`` over their requests' rows ``[pages, page_size, d]``,
-    whose first ``value_dim`` columns are the values; result ``[N, heads, value_dim]``.
+    whose first ``value_dim`` columns are the values; result ``[N, heads, value_dim]``.  ``sink`` (float32 ``[heads]``): a further
+    term ``exp(sink[head])`` in every softmax sum that belongs to no key.
 
     bfloat16 with both widths in steps of 16: the mma.sync kernel (prompt portions and single tokens alike: a tile is up to
     ``64 // heads`` consecutive tokens of one request times the heads).  float32, and every other size: the CUDA-core kernel."""
@@ -59,7 +60,9 @@ def latent_attention(q: torch.Tensor, pool: torch.Tensor, ctx: Any, table: torch
     rot = d - value_dim
     if BACKEND != "mma" or q.dtype != torch.bfloat16 or not supported(value_dim, rot):
         return F.paged_attention_simt_latent(q, pool, value_dim=value_dim, positions=ctx.positions, token_entry=ctx.token_entry,
-                                             block_table=table, scale=scale, window=window)
+                                             block_table=table, scale=scale, window=window, sink=sink)
+    if sink is not None:
+        native.require(sink, "sink", dtype=torch.float32, shape=(heads,))
     per_tile = max(1, ROWS_PER_TILE // heads)
     decode = ctx.all_decode and n == ctx.num_entries
     maps = ctx.__dict__.setdefault("_tile_maps", {})
@@ -78,7 +81,7 @@ def latent_attention(q: torch.Tensor, pool: torch.Tensor, ctx: Any, table: torch
             floats = n * heads * splits * (value_dim + 2)
             scratch = torch.empty(floats, dtype=torch.float32, device=q.device)
     native.call("b200_attention_latent_bf16", q.data_ptr(), pool.data_ptr(), out.data_ptr(), ctx.positions.data_ptr(), table.data_ptr(),
-                table.shape[1], pool.shape[1], heads, float(scale), int(window), tiles[0].data_ptr(), tiles[1].data_ptr(),
+                table.shape[1], pool.shape[1], heads, float(scale), int(window), native.ptr(sink), tiles[0].data_ptr(), tiles[1].data_ptr(),
                 tiles[2].data_ptr(), count, splits, native.ptr(scratch), floats, native.stream_ptr(),
                 library=library_name(value_dim, rot), launches=2 if splits > 1 else 1)
     return out

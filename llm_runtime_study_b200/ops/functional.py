@@ -82,7 +82,10 @@ def linear_f32(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | None 
     return out
 
 
-def silu_mul(gate_up: torch.Tensor) -> torch.Tensor:
+GATE_ACTS = {"silu": 1, "gelu_tanh": 2}     # as numbered in csrc/common.cuh
+
+
+def silu_mul(gate_up: torch.Tensor, act: str = "silu") -> torch.Tensor:
     """``silu(gate) * up`` for rows laid out as ``[gate | up]``."""
 
     require(gate_up, "gate_up", dims=2)
@@ -90,12 +93,12 @@ def silu_mul(gate_up: torch.Tensor) -> torch.Tensor:
     if two_i % 2:
         raise KernelError("silu_mul: row width must be even ([gate | up])")
     out = torch.empty((n, two_i // 2), dtype=gate_up.dtype, device=gate_up.device)
-    call("b200_silu_mul", ptr(gate_up), ptr(out), n, two_i // 2, tag(gate_up.dtype), stream_ptr())
+    call("b200_silu_mul", ptr(gate_up), ptr(out), n, two_i // 2, GATE_ACTS[act], tag(gate_up.dtype), stream_ptr())
     return out
 
 
-def silu_mul_interleaved(gate_up: torch.Tensor) -> torch.Tensor:
-    """``silu(gate) * up`` for rows laid out in blocks of eight, ``[g0..g7 | u0..u7 | g8..g15 | ...]``
+def silu_mul_interleaved(gate_up: torch.Tensor, act: str = "silu") -> torch.Tensor:
+    """``silu(gate) * up`` (or another gate) for rows laid out in blocks of eight, ``[g0..g7 | u0..u7 | g8..g15 | ...]``
     (the layout of a stacked gate/up projection whose kernels can apply the activation themselves)."""
 
     require(gate_up, "gate_up", dims=2)
@@ -103,7 +106,7 @@ def silu_mul_interleaved(gate_up: torch.Tensor) -> torch.Tensor:
     if two_i % 16:
         raise KernelError("silu_mul_interleaved: row width must be a multiple of 16")
     out = torch.empty((n, two_i // 2), dtype=gate_up.dtype, device=gate_up.device)
-    call("b200_silu_mul_interleaved", ptr(gate_up), ptr(out), n, two_i // 2, tag(gate_up.dtype), stream_ptr())
+    call("b200_silu_mul_interleaved", ptr(gate_up), ptr(out), n, two_i // 2, GATE_ACTS[act], tag(gate_up.dtype), stream_ptr())
     return out
 
 
@@ -211,11 +214,12 @@ def qk_rownorm_write(
 def paged_attention_simt_rules(
     q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, *, positions: torch.Tensor, token_entry: torch.Tensor,
     block_table: torch.Tensor, scale: float, window: int = 0, softcap: float = 0.0, slopes: torch.Tensor | None = None,
-    sink: bool = False, chunk: int = 0, log_bias: tuple[torch.Tensor, torch.Tensor] | None = None,
+    sink: "bool | torch.Tensor" = False, chunk: int = 0, log_bias: tuple[torch.Tensor, torch.Tensor] | None = None,
 ) -> torch.Tensor:
     """``paged_attention_simt`` with rules on the scores: ``S <- cap * tanh(S / cap)`` (``softcap > 0``), then
     ``S <- S - slopes[head] * (p - t)``, ``S <- S - r1[head] * ln(1 + r2[head] * (p - t))`` (``log_bias = (r1, r2)``), and with
-    ``sink`` the weights ``exp(S) / (1 + sum exp(S))``.  ``chunk > 0``: position p sees t only inside its own block of ``chunk``
+    ``sink`` the weights ``exp(S) / (1 + sum exp(S))``, or, with one number per query head (float32 ``[nq]``),
+    ``exp(S) / (exp(sink[head]) + sum exp(S))``.  ``chunk > 0``: position p sees t only inside its own block of ``chunk``
     positions (counted from 0).  Values may have a head size of their own: q ``[N, nq, d]``, keys ``[pages, nkv, page, d]``,
     values ``[pages, nkv, page, dv]``, result ``[N, nq, dv]``."""
 
@@ -237,12 +241,15 @@ def paged_attention_simt_rules(
         r1, r2 = log_bias
         require(r1, "log_bias[0]", dtype=torch.float32, shape=(nq,))
         require(r2, "log_bias[1]", dtype=torch.float32, shape=(nq,))
+    sinks = None
+    if isinstance(sink, torch.Tensor):
+        sinks, sink = require(sink, "sink", dtype=torch.float32, shape=(nq,)), False
     if d > 256 or dv > 256:
         raise KernelError(f"head sizes {d} and {dv} must be at most 256")
     out = torch.empty((n, nq, dv), dtype=q.dtype, device=q.device)
     call("b200_paged_attention_simt_masked", ptr(q), ptr(k_pool), ptr(v_pool), ptr(out), ptr(positions), ptr(token_entry),
          ptr(block_table), block_table.shape[1], page_size, n, nq, nkv, d, dv, dv, float(scale), int(window), float(softcap),
-         ptr(slopes), 1 if sink else 0, int(chunk), ptr(r1), ptr(r2), tag(q.dtype), stream_ptr())
+         ptr(slopes), 1 if sink else 0, int(chunk), ptr(r1), ptr(r2), ptr(sinks), tag(q.dtype), stream_ptr())
     return out
 
 
@@ -255,13 +262,23 @@ def relu2(x: torch.Tensor) -> torch.Tensor:
     return out
 
 
+def soft_cap(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """``x <- cap * tanh(x / cap)`` in place on float32 values; ``x`` is returned."""
+
+    require(x, "x", dtype=torch.float32)
+    call("b200_soft_cap", ptr(x), x.numel(), float(cap), stream_ptr())
+    return x
+
+
 def embedding_sum(ids: torch.Tensor, table: torch.Tensor, bigram: torch.Tensor | None, *, positions: torch.Tensor,
                   token_entry: torch.Tensor, q_start: torch.Tensor, slots: torch.Tensor, previous: torch.Tensor | None,
-                  freq: torch.Tensor | None, buckets: int = 0, mul_prev: int = 0, mul_cur: int = 0, scale: float = 1.0) -> torch.Tensor:
+                  freq: torch.Tensor | None, buckets: int = 0, mul_prev: int = 0, mul_cur: int = 0, scale: float = 1.0,
+                  norm: "tuple[torch.Tensor, float] | None" = None, rounded_dtype: torch.dtype | None = None):
     """``table[id] * scale + bigram[row] + pos(p)`` as float32 rows: ``row = (previous token * mul_prev + id * mul_cur) mod buckets``,
     row ``buckets`` at position 0; ``pos(p)``: column ``2i`` is ``sin(p * freq[i])``, column ``2i + 1`` the cosine (``freq`` float64).
     The token before a step's first token of a request is read from ``previous[slot]`` (int32 per request slot), which then
-    receives the entry's last token.  ``bigram`` and ``freq`` may each be ``None``."""
+    receives the entry's last token.  ``bigram`` and ``freq`` may each be ``None``.  ``norm = (weight, eps)``: the sum is
+    RMS-normed in the same launch, and with ``rounded_dtype`` (the table's type) ``(rows, the rows in that type)`` is returned."""
 
     require(ids, "ids", dtype=torch.int32, dims=1)
     require(table, "table", dims=2)
@@ -276,11 +293,17 @@ def embedding_sum(ids: torch.Tensor, table: torch.Tensor, bigram: torch.Tensor |
         require(previous, "previous", dtype=torch.int32)
     if freq is not None:
         require(freq, "freq", dtype=torch.float64, shape=((hidden + 1) // 2,))
+    weight, eps = norm if norm is not None else (None, 0.0)
+    if weight is not None:
+        require(weight, "norm weight", dtype=torch.float32, shape=(hidden,))
+    if rounded_dtype is not None and (weight is None or rounded_dtype != table.dtype):
+        raise KernelError("embedding_sum rounds normed rows only, to the table's type")
     out = torch.empty((n, hidden), dtype=torch.float32, device=ids.device)
+    rounded = None if rounded_dtype is None else torch.empty((n, hidden), dtype=rounded_dtype, device=ids.device)
     call("b200_embedding_sum", ptr(ids), ptr(table), ptr(bigram), ptr(out), ptr(positions), ptr(token_entry), ptr(q_start), ptr(slots),
-         ptr(previous), ptr(freq), n, entries, hidden, vocab, int(buckets), int(mul_prev), int(mul_cur), float(scale), tag(table.dtype),
-         stream_ptr())
-    return out
+         ptr(previous), ptr(freq), n, entries, hidden, vocab, int(buckets), int(mul_prev), int(mul_cur), float(scale), ptr(weight),
+         float(eps), ptr(rounded), tag(table.dtype), stream_ptr())
+    return out if rounded is None else (out, rounded)
 
 
 def glu_limit(gate_up: torch.Tensor, limit: float, alpha: float) -> torch.Tensor:
@@ -327,11 +350,12 @@ def add_rows(resid: torch.Tensor, a: torch.Tensor | None = None, b: torch.Tensor
 
 def paged_attention_simt_latent(
     q: torch.Tensor, pool: torch.Tensor, *, value_dim: int, positions: torch.Tensor, token_entry: torch.Tensor,
-    block_table: torch.Tensor, scale: float, window: int = 0,
+    block_table: torch.Tensor, scale: float, window: int = 0, sink: torch.Tensor | None = None,
 ) -> torch.Tensor:
     """Causal attention of every query head over one shared row per token whose leading ``value_dim`` columns are also the
     value: q ``[N, heads, d]``, pool ``[pages, page_size, d]``, result ``[N, heads, value_dim]``.  32-bit arithmetic, tiles
-    of 32 keys from key 0 of the window's first tile, so the order of every sum depends on the token's position alone."""
+    of 32 keys from key 0 of the window's first tile, so the order of every sum depends on the token's position alone.
+    ``sink`` (float32 ``[heads]``): a further term ``exp(sink[head])`` in every sum that belongs to no key."""
 
     require(q, "q", dims=3)
     n, nq, d = q.shape
@@ -343,7 +367,9 @@ def paged_attention_simt_latent(
     require(token_entry, "token_entry", dtype=torch.int32, shape=(n,))
     require(block_table, "block_table", dtype=torch.int32, dims=2)
     out = torch.empty((n, nq, value_dim), dtype=q.dtype, device=q.device)
-    call("b200_paged_attention_simt_strided", ptr(q), ptr(pool), ptr(pool), ptr(out), ptr(positions), ptr(token_entry),
+    if sink is not None:
+        require(sink, "sink", dtype=torch.float32, shape=(nq,))
+    call("b200_paged_attention_simt_masked", ptr(q), ptr(pool), ptr(pool), ptr(out), ptr(positions), ptr(token_entry),
          ptr(block_table), block_table.shape[1], page_size, n, nq, 1, d, value_dim, d, float(scale), int(window), 0.0, None, 0,
-         tag(q.dtype), stream_ptr())
+         0, None, None, ptr(sink), tag(q.dtype), stream_ptr())
     return out

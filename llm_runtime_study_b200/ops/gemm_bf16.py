@@ -8,6 +8,7 @@ import torch
 
 from ..errors import KernelError
 from . import native
+from .functional import GATE_ACTS
 from .native import c_int, c_void_p
 
 native.register_library(
@@ -115,14 +116,20 @@ def few_rows_kernel(m: int, n: int, k: int) -> str:
     return "splitk" if k >= 16384 and n * k >= SKINNY_LARGE else "skinny"
 
 
+def gated_unit(swiglu: "bool | str") -> int:
+    """The kernels' number of a gated unit: 0 for none, else its gate (``True``: SiLU)."""
+
+    return 0 if not swiglu else GATE_ACTS["silu" if swiglu is True else swiglu]
+
+
 def linear(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | None = None,
-           out_dtype: torch.dtype = torch.bfloat16, *, swiglu: bool = False, add_to: torch.Tensor | None = None,
+           out_dtype: torch.dtype = torch.bfloat16, *, swiglu: "bool | str" = False, add_to: torch.Tensor | None = None,
            kernel: str | None = None, tile_n: int | None = None, splits: int = 0, stages: int = 0) -> torch.Tensor:
     """``x @ weight.T (+ bias)`` on the tcgen05 tensor cores; float32 accumulation; bfloat16 or
     float32 output.
 
     ``swiglu``: the weight holds gate and up rows interleaved in blocks of eight and the result is
-    ``silu(gate) * up``, half as wide.  ``add_to`` (float32 ``[M, N]``): the product is added to it
+    ``silu(gate) * up``, half as wide (``"gelu_tanh"``: with that gate).  ``add_to`` (float32 ``[M, N]``): the product is added to it
     in place and it is returned.  ``kernel``: "persistent" (one CTA per tile of 128 rows and
     ``tile_n`` = 128 or 256 columns), "pair" (two CTAs per 256 x 256 tile), "streamk" (few
     tiles: up to three SMs share a tile's K range) or "splitk" (few rows: a cluster of ``splits``
@@ -162,7 +169,7 @@ def linear(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | None = No
                               "256 columns, or 128 with the persistent kernel")
     partials, flags = _streamk_workspace(x.device) if kernel == "streamk" else (None, None)
     native.call("b200_gemm_tcgen05", x.data_ptr(), weight.data_ptr(), native.ptr(bias), out.data_ptr(), m, n, k,
-                out.shape[1], 1 if out_dtype == torch.float32 else 0, 1 if swiglu else 0, 0 if add_to is None else 1,
+                out.shape[1], 1 if out_dtype == torch.float32 else 0, gated_unit(swiglu), 0 if add_to is None else 1,
                 KERNELS[kernel], tile_n, splits, stages, native.ptr(partials), native.ptr(flags), native.stream_ptr())
     return out
 
@@ -183,7 +190,7 @@ def check_error() -> None:
 
 
 def linear_skinny(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | None = None,
-                  out_dtype: torch.dtype = torch.bfloat16, *, variant: int = 0, swiglu: bool = False,
+                  out_dtype: torch.dtype = torch.bfloat16, *, variant: int = 0, swiglu: "bool | str" = False,
                   row_scale: torch.Tensor | None = None) -> torch.Tensor:
     """``x @ weight.T (+ bias)`` for at most 16 rows of ``x``: the weight-streaming kernel.
     ``swiglu``: see ``linear``.  ``row_scale`` (float32 ``[16]``): the rows of ``x`` still lack these factors
@@ -206,7 +213,7 @@ def linear_skinny(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | No
     width = n // 2 if swiglu else n
     out = torch.empty((m, width), dtype=out_dtype, device=x.device)
     native.call("b200_gemm_skinny_variant", x.data_ptr(), weight.data_ptr(), native.ptr(bias), out.data_ptr(), m, n, k, width,
-                1 if out_dtype == torch.float32 else 0, variant, 1 if swiglu else 0, native.ptr(row_scale), native.stream_ptr())
+                1 if out_dtype == torch.float32 else 0, variant, gated_unit(swiglu), native.ptr(row_scale), native.stream_ptr())
     return out
 
 

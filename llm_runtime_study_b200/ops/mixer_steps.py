@@ -65,12 +65,12 @@ def latent_prepare(
     rows: torch.Tensor, *, q_offset: int, q_rank: int, q_weight: torch.Tensor, eps: float, positions: torch.Tensor,
     token_entry: torch.Tensor, kv_offset: int = 0, kv_rank: int = 0, kv_weight: torch.Tensor | None = None, rot: int = 0,
     rot_dims: int = 0, inv_freq: torch.Tensor | None = None, block_table: torch.Tensor | None = None, page_size: int = 0,
-    pool: torch.Tensor | None = None,
+    pool: torch.Tensor | None = None, interleaved: bool = False, rot_factor: float = 1.0,
 ) -> torch.Tensor:
     """From rows of a stacked projection: columns ``q_offset .. + q_rank`` RMS-normed with ``q_weight`` are returned
     ``[N, q_rank]``; with ``kv_rank > 0`` columns ``kv_offset .. + kv_rank`` RMS-normed with ``kv_weight`` and the ``rot``
-    columns behind them (the first ``rot_dims`` rotated by the position, pairs ``(i, i + rot_dims/2)``) are written into
-    the pages ``[pages, page_size, kv_rank + rot]``."""
+    columns behind them (the first ``rot_dims`` rotated by the position, pairs ``(i, i + rot_dims/2)`` or, ``interleaved``,
+    ``(2i, 2i + 1)``; cosine and sine times ``rot_factor``) are written into the pages ``[pages, page_size, kv_rank + rot]``."""
 
     require(rows, "rows", dims=2)
     n, ld = rows.shape
@@ -90,15 +90,16 @@ def latent_prepare(
             require(inv_freq, "inv_freq", dtype=torch.float32, shape=(rot_dims // 2,))
     out = torch.empty((n, q_rank), dtype=dt, device=rows.device)
     call("b200_latent_prepare", ptr(rows), ld, q_offset, q_rank, ptr(q_weight), ptr(out), kv_offset, kv_rank, ptr(kv_weight), rot,
-         rot_dims, ptr(inv_freq), float(eps), ptr(positions), ptr(token_entry), ptr(block_table), stride, page_size, ptr(pool), n,
+         rot_dims, ptr(inv_freq), 1 if interleaved else 0, float(rot_factor), float(eps), ptr(positions), ptr(token_entry), ptr(block_table), stride, page_size, ptr(pool), n,
          tag(dt), stream_ptr())
     return out
 
 
 def rope_slice(src: torch.Tensor, dst: torch.Tensor, *, heads: int, src_head: int, src_offset: int, dst_head: int,
-               dst_offset: int, rot: int, rot_dims: int, inv_freq: torch.Tensor, positions: torch.Tensor) -> None:
+               dst_offset: int, rot: int, rot_dims: int, inv_freq: torch.Tensor, positions: torch.Tensor, interleaved: bool = False,
+               rot_factor: float = 1.0) -> None:
     """Columns ``src_offset .. + rot`` of every head of ``src`` (``[N, heads * src_head]``), the first ``rot_dims`` of them
-    rotated by the token's position, are written to columns ``dst_offset ..`` of every head of ``dst``."""
+    rotated by the token's position (see ``latent_prepare``), are written to columns ``dst_offset ..`` of every head of ``dst``."""
 
     require(src, "src", dims=2)
     require(dst, "dst", dtype=src.dtype, dims=2)
@@ -109,7 +110,7 @@ def rope_slice(src: torch.Tensor, dst: torch.Tensor, *, heads: int, src_head: in
     if src.shape[1] < heads * src_head or dst.shape[1] < heads * dst_head or dst.shape[0] != n:
         raise KernelError("rope_slice: the heads do not fit the rows")
     call("b200_rope_slice", ptr(src), src.shape[1], src_head, src_offset, ptr(dst), dst.shape[1], dst_head, dst_offset, heads, rot,
-         rot_dims, ptr(inv_freq), ptr(positions), n, tag(src.dtype), stream_ptr())
+         rot_dims, ptr(inv_freq), 1 if interleaved else 0, float(rot_factor), ptr(positions), n, tag(src.dtype), stream_ptr())
 
 
 def sigmoid_gate(x: torch.Tensor, gate_rows: torch.Tensor, *, gate_offset: int, group: int) -> torch.Tensor:
@@ -128,8 +129,8 @@ def sigmoid_gate(x: torch.Tensor, gate_rows: torch.Tensor, *, gate_offset: int, 
 
 
 def norm_accumulate_round(x: "torch.Tensor | PairedRows | None", weight: torch.Tensor | None, eps: float, resid: torch.Tensor,
-                          rounded_dtype: torch.dtype | None) -> torch.Tensor | None:
-    """``resid += x * rsqrt(mean(x^2) + eps) * weight`` in place on float32 rows (nothing is added when ``x`` is ``None``);
+                          rounded_dtype: torch.dtype | None, factor: float = 1.0) -> torch.Tensor | None:
+    """``resid += factor * x * rsqrt(mean(x^2) + eps) * weight`` in place on float32 rows (nothing is added when ``x`` is ``None``);
     with ``rounded_dtype`` the updated rows are also returned in that type, for the sublayer that reads them next.  ``x`` may be
     ``PairedRows``: then row ``t`` of the sublayer's output is ``sum_j weights[t, j] * rows[pair_row[t, j]]``, formed inside the
     kernel.  The width is at most 12,288 (a row is kept in shared memory)."""
@@ -152,7 +153,7 @@ def norm_accumulate_round(x: "torch.Tensor | PairedRows | None", weight: torch.T
         rounded = torch.empty((n, hidden), dtype=rounded_dtype, device=resid.device)
     if x is None and rounded is None:
         return None
-    call("b200_norm_accumulate_round", ptr(x), ptr(weight), ptr(resid), ptr(rounded), n, hidden, float(eps), ptr(pair_row), ptr(pair_w),
+    call("b200_norm_accumulate_round", ptr(x), ptr(weight), ptr(resid), ptr(rounded), n, hidden, float(eps), float(factor), ptr(pair_row), ptr(pair_w),
          top, tag(rounded_dtype or torch.float32), stream_ptr())
     return rounded
 

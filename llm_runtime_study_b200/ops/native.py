@@ -38,8 +38,8 @@ _LIBRARIES = {
             "b200_embedding_weighted": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float,
                                         c_float, c_int, c_void_p],
             "b200_add_rmsnorm": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_int, c_void_p],
-            "b200_silu_mul": [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
-            "b200_silu_mul_interleaved": [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+            "b200_silu_mul": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+            "b200_silu_mul_interleaved": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
             "b200_qk_norm_rope_write": [
                 c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p,
                 c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
@@ -52,12 +52,13 @@ _LIBRARIES = {
             "b200_rmsnorm_accumulate": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_int, c_void_p],
             "b200_add_rows": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
             "b200_relu2": [c_void_p, c_void_p, c_longlong, c_int, c_void_p],
+            "b200_soft_cap": [c_void_p, c_longlong, c_float, c_void_p],
         },
     ),
     "b200_embedding_sum": (
         ("embedding_sum.cu",),
         {"b200_embedding_sum": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                                c_int, c_int, c_int, c_int, c_int, c_longlong, c_longlong, c_float, c_int, c_void_p]},
+                                c_int, c_int, c_int, c_int, c_int, c_longlong, c_longlong, c_float, c_void_p, c_float, c_void_p, c_int, c_void_p]},
     ),
     "b200_mingru": (
         ("mingru.cu",),
@@ -84,8 +85,8 @@ _LIBRARIES = {
             ],
             "b200_paged_attention_simt_masked": [
                 c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_float, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int,
-                c_void_p,
+                c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_float, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p,
+                c_int, c_void_p,
             ],
             "b200_paged_attention_simt_strided": [
                 c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
@@ -98,16 +99,23 @@ _LIBRARIES = {
         {
             "b200_linear_scan": [
                 c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p,
-                c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
+                c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p,
             ],
+            "b200_linear_scan_row_gates": [
+                c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p,
+            ],
+            "b200_memory_gates": [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p,
+                                  c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+            "b200_channel_decay": [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_void_p],
             "b200_delta_prepare": [
                 c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                 c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                 c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_void_p,
             ],
             "b200_conv_state_update": [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p],
-            "b200_group_norm_gate": [c_void_p, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_int, c_void_p,
-                                     c_void_p, c_int, c_void_p],
+            "b200_group_norm_gate": [c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_float, c_void_p, c_void_p, c_float, c_void_p,
+                                     c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p],
         },
     ),
     "b200_mixer_steps": (
@@ -118,11 +126,12 @@ _LIBRARIES = {
             "b200_head_norm_write_at": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_int, c_void_p, c_void_p, c_void_p,
                                         c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
             "b200_latent_prepare": [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int,
-                                    c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p],
+                                    c_void_p, c_int, c_float, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int,
+                                    c_void_p],
             "b200_rope_slice": [c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
-                                c_void_p, c_int, c_int, c_void_p],
+                                c_int, c_float, c_void_p, c_int, c_int, c_void_p],
             "b200_sigmoid_gate": [c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
-            "b200_norm_accumulate_round": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p, c_int,
+            "b200_norm_accumulate_round": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_void_p, c_void_p, c_int,
                                            c_int, c_void_p],
         },
     ),

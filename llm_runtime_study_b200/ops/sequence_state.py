@@ -13,13 +13,15 @@ from .native import call, ptr, require, stream_ptr, tag
 def linear_scan(
     q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, *, heads: int, qk_heads: int, dim: int, vdim: int,
     state: torch.Tensor, q_start: torch.Tensor, slots: torch.Tensor, gate: torch.Tensor | None = None,
-    decay: torch.Tensor | None = None, beta: torch.Tensor | None = None, silu: bool = False, fixed_order: bool = False,
+    decay: torch.Tensor | None = None, beta: torch.Tensor | None = None, silu: bool = False, q_scale: float = 1.0,
+    fixed_order: bool = False,
 ) -> torch.Tensor:
     """Per request (entry ``e`` owns rows ``q_start[e] .. q_start[e+1]-1`` and the state row ``slots[e]``) and head,
     token after token: ``S <- D S + k u^T``, ``o = S^T q`` with ``D`` the head's constant ``decay`` or the row's
     ``gate`` factors (one per key channel), and ``u = v`` or, with ``beta``, ``beta (v - (D S)^T k)``.  ``q`` and
     ``k`` are ``[N, qk_heads * dim]`` column blocks (a row stride of their own is fine), ``v`` ``[N, heads * vdim]``;
-    head ``h`` reads q/k head ``h // (heads / qk_heads)``.  ``silu`` applies SiLU to q, k and v as they are read.
+    head ``h`` reads q/k head ``h // (heads / qk_heads)``.  ``silu`` applies SiLU to q, k and v as they are read;
+    q is multiplied by ``q_scale`` then.
     ``state`` is ``[slots, heads, dim, vdim]`` float32 and is updated in place.  ``fixed_order``: every sum is formed in
     an order that does not depend on the shape of the batch (the kernel otherwise spreads a column over more lanes when few
     requests bring long portions), so a token's bits do not depend on the cut.  Returns float32 ``[N, heads * vdim]``."""
@@ -45,8 +47,82 @@ def linear_scan(
     out = torch.empty((n, heads * vdim), dtype=torch.float32, device=q.device)
     call("b200_linear_scan", ptr(q), ptr(k), ptr(v), q.stride(0), k.stride(0), v.stride(0), ptr(gate), heads * dim, ptr(decay),
          ptr(beta), heads, ptr(state), ptr(out), heads * vdim, ptr(q_start), ptr(slots), entries, n, heads, qk_heads, dim, vdim,
-         1 if silu else 0, 1 if fixed_order else 0, tag(q.dtype), stream_ptr())
+         1 if silu else 0, float(q_scale), 1 if fixed_order else 0, tag(q.dtype), stream_ptr())
     return out
+
+
+def linear_scan_row_gates(
+    q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, *, heads: int, dim: int, vdim: int, decay: torch.Tensor, gain: torch.Tensor,
+    state: torch.Tensor, norm_state: torch.Tensor, q_start: torch.Tensor, slots: torch.Tensor, q_scale: float = 1.0,
+    fixed_order: bool = False,
+) -> tuple[torch.Tensor, torch.Tensor]:
+    """``linear_scan`` with one decay and one input gain per row and head, and a normaliser: ``S <- decay S + gain k v^T``,
+    ``n <- decay n + gain k``; returns ``S^T q`` float32 ``[N, heads * vdim]`` and ``n . q`` float32 ``[N, heads]`` (q times
+    ``q_scale`` as it is read).  ``state`` ``[slots, heads, dim, vdim]`` and ``norm_state`` ``[slots, heads, dim]`` float32 are
+    updated in place; ``decay`` and ``gain`` are float32 ``[N, heads]``.  ``fixed_order`` as for ``linear_scan``."""
+
+    n = q.shape[0]
+    for t, name, width in ((q, "q", heads * dim), (k, "k", heads * dim), (v, "v", heads * vdim)):
+        if t.device.type != "cuda" or t.dim() != 2 or t.shape != (n, width) or t.stride(1) != 1 or t.dtype != q.dtype:
+            raise KernelError(f"{name} must be CUDA rows [{n}, {width}] of one type with unit column stride")
+    require(state, "state", dtype=torch.float32, dims=4)
+    require(norm_state, "norm_state", dtype=torch.float32, dims=3)
+    if tuple(state.shape[1:]) != (heads, dim, vdim) or tuple(norm_state.shape[1:]) != (heads, dim) or norm_state.shape[0] != state.shape[0]:
+        raise KernelError(f"states have shapes {tuple(state.shape)} and {tuple(norm_state.shape)}, expected [slots, {heads}, {dim}, {vdim}] "
+                          f"and [slots, {heads}, {dim}]")
+    require(decay, "decay", dtype=torch.float32, shape=(n, heads))
+    require(gain, "gain", dtype=torch.float32, shape=(n, heads))
+    require(q_start, "q_start", dtype=torch.int32, dims=1)
+    entries = q_start.shape[0] - 1
+    require(slots, "slots", dtype=torch.int32, shape=(entries,))
+    out = torch.empty((n, heads * vdim), dtype=torch.float32, device=q.device)
+    norm_out = torch.empty((n, heads), dtype=torch.float32, device=q.device)
+    call("b200_linear_scan_row_gates", ptr(q), ptr(k), ptr(v), q.stride(0), k.stride(0), v.stride(0), ptr(decay), ptr(gain), ptr(state),
+         ptr(norm_state), ptr(out), ptr(norm_out), ptr(q_start), ptr(slots), entries, n, heads, dim, vdim, float(q_scale),
+         1 if fixed_order else 0, tag(q.dtype), stream_ptr())
+    return out, norm_out
+
+
+def memory_gates(
+    proj: torch.Tensor, *, heads: int, i_offset: int, f_offset: int, i_bias: torch.Tensor, f_bias: torch.Tensor, cap: float,
+    m_state: torch.Tensor, q_start: torch.Tensor, slots: torch.Tensor,
+) -> tuple[torch.Tensor, torch.Tensor, torch.Tensor]:
+    """Exponential gates kept in range by a running maximum.  With ``i = cap tanh((zi + i_bias) / cap)`` and
+    ``f = ln sigmoid(cap tanh((zf + f_bias) / cap))`` (logits: columns ``i_offset + h`` and ``f_offset + h`` of ``proj``), token after
+    token: ``m_t = max(f + m_(t-1), i)`` from the slot's ``m`` (``m_state`` float32 ``[slots, heads]``, updated in place).  Returns
+    float32 ``[N, heads]`` each: ``exp(f + m_(t-1) - m_t)``, ``exp(i - m_t)`` and ``exp(-m_t)``."""
+
+    require(proj, "proj", dims=2)
+    n, ld = proj.shape
+    require(i_bias, "i_bias", dtype=torch.float32, shape=(heads,))
+    require(f_bias, "f_bias", dtype=torch.float32, shape=(heads,))
+    require(m_state, "m_state", dtype=torch.float32, dims=2)
+    if m_state.shape[1] != heads or max(i_offset, f_offset) + heads > ld:
+        raise KernelError("memory_gates: the logits lie outside the rows, or the state has another number of heads")
+    require(q_start, "q_start", dtype=torch.int32, dims=1)
+    entries = q_start.shape[0] - 1
+    require(slots, "slots", dtype=torch.int32, shape=(entries,))
+    decay, gain, floor = torch.empty((3, n, heads), dtype=torch.float32, device=proj.device)
+    call("b200_memory_gates", ptr(proj), ld, i_offset, f_offset, ptr(i_bias), ptr(f_bias), float(cap), ptr(m_state), ptr(decay), ptr(gain),
+         ptr(floor), ptr(q_start), ptr(slots), entries, heads, tag(proj.dtype), stream_ptr())
+    return decay, gain, floor
+
+
+def channel_decay(proj: torch.Tensor, up: torch.Tensor, bias: torch.Tensor, *, offset: int, tau: float) -> torch.Tensor:
+    """Decays per key channel from a low-rank map: ``sigmoid(proj[:, offset : offset + rank] @ up + bias)^(1 / tau)``, float32
+    ``[N, width]``; ``up`` is ``[rank, width]`` (the map's weight transposed) in the type of ``proj``."""
+
+    require(proj, "proj", dims=2)
+    n, ld = proj.shape
+    require(up, "up", dtype=proj.dtype, dims=2)
+    rank, width = up.shape
+    require(bias, "bias", dtype=torch.float32, shape=(width,))
+    if offset + rank > ld:
+        raise KernelError("channel_decay: the low-rank columns lie outside the rows")
+    alpha = torch.empty((n, width), dtype=torch.float32, device=proj.device)
+    call("b200_channel_decay", ptr(proj), ld, offset, rank, ptr(up), ptr(bias), float(tau), ptr(alpha), n, width, tag(proj.dtype),
+         stream_ptr())
+    return alpha
 
 
 def delta_prepare(
@@ -100,18 +176,29 @@ def conv_state_update(proj: torch.Tensor, conv_state: torch.Tensor, q_start: tor
 
 
 def group_norm_gate(x: torch.Tensor, weight: torch.Tensor, eps: float, gate_in: torch.Tensor, *, gate_offset: int = 0,
-                    gate_up: torch.Tensor | None = None, out_dtype: torch.dtype) -> torch.Tensor:
-    """``x`` float32 ``[N, width]`` in groups of ``len(weight)`` columns: each group divided by its root mean square,
-    times ``weight``, times ``sigmoid(logit)``; the logits are columns ``gate_offset ..`` of ``gate_in`` (``width`` of
+                    gate_up: torch.Tensor | None = None, out_dtype: torch.dtype, group: int | None = None, act: str = "sigmoid",
+                    divisor: "tuple[torch.Tensor, torch.Tensor, float] | None" = None) -> torch.Tensor:
+    """``x`` float32 ``[N, width]`` in groups of ``group`` columns (default ``len(weight)``): each group divided by its root mean
+    square, times ``weight`` (one group's, or ``[width]``), times ``sigmoid(logit)`` or ``silu(logit)`` (``act``).  ``divisor =
+    (den, floor, e)``: before that, each group divided by ``max(|den|, floor) + e`` with its own numbers (float32 ``[N, width /
+    group]`` each).  The logits are columns ``gate_offset ..`` of ``gate_in`` (``width`` of
     them), or, with ``gate_up`` ``[rank, width]`` (a low-rank map's weight transposed),
     ``gate_in[:, gate_offset : gate_offset + rank] @ gate_up``."""
 
     require(x, "x", dtype=torch.float32, dims=2)
     n, width = x.shape
     require(weight, "weight", dtype=torch.float32, dims=1)
-    group = weight.shape[0]
-    if width % group:
-        raise KernelError(f"width {width} is not a multiple of the group size {group}")
+    group = weight.shape[0] if group is None else group
+    if group <= 0 or width % group or weight.shape[0] not in (group, width):
+        raise KernelError(f"width {width} is not a multiple of the group size {group}, or the weight has {weight.shape[0]} entries")
+    if act not in ("sigmoid", "silu"):
+        raise KernelError(f"unknown gate {act!r}")
+    den = floor = None
+    den_eps = 0.0
+    if divisor is not None:
+        den, floor, den_eps = divisor
+        require(den, "divisor", dtype=torch.float32, shape=(n, width // group))
+        require(floor, "divisor floor", dtype=torch.float32, shape=(n, width // group))
     require(gate_in, "gate_in", dtype=out_dtype, dims=2)
     rank = 0
     if gate_up is not None:
@@ -123,6 +210,6 @@ def group_norm_gate(x: torch.Tensor, weight: torch.Tensor, eps: float, gate_in: 
         raise KernelError("group_norm_gate: the gate's columns lie outside gate_in")
     out = torch.empty((n, width), dtype=out_dtype, device=x.device)
     gate_ptr = gate_in.data_ptr() + gate_offset * gate_in.element_size()
-    call("b200_group_norm_gate", ptr(x), n, width, group, ptr(weight), float(eps), gate_ptr, gate_in.shape[1], rank,
-         ptr(gate_up), ptr(out), tag(out_dtype), stream_ptr())
+    call("b200_group_norm_gate", ptr(x), n, width, group, ptr(weight), weight.shape[0], float(eps), ptr(den), ptr(floor), float(den_eps),
+         gate_ptr, gate_in.shape[1], rank, ptr(gate_up), 1 if act == "silu" else 0, ptr(out), tag(out_dtype), stream_ptr())
     return out

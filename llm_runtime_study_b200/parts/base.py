@@ -150,6 +150,15 @@ class PositionEncoding(Part):
     def rotary_parameters(self) -> tuple[torch.Tensor, int] | None:
         return None
 
+    def rotary_layout(self) -> tuple[torch.Tensor, int, bool, float]:
+        """``(inv_freq, rotary_dim, interleaved, factor)`` for kernels that take either pairing of the rotated columns
+        (``(2i, 2i + 1)`` when interleaved, else ``(i, i + rotary_dim / 2)``) and a factor on cosine and sine."""
+
+        parameters = self.rotary_parameters()
+        if parameters is None:
+            raise NotImplementedError("this position encoding is not a rotation of pairs of columns")
+        return (*parameters, False, 1.0)
+
     def apply(self, q: torch.Tensor, k: torch.Tensor | None, ctx: Any) -> None:
         """Rotate/shift ``q`` and ``k`` in place (only called when
         ``rotary_parameters()`` is ``None``)."""

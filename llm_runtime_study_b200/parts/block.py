@@ -88,14 +88,16 @@ class OutputNormBlock(Block):
     """``h = h + norm_1(mixer(h)); h = h + norm_2(ffn(h))``: the sublayers read the residual rows themselves (rounded to
     the activation type where that is not float32) and the norm sits on their output only.  The kernel that normalises a
     sublayer's output adds it into the float32 rows and hands the next sublayer its rounded copy in the same pass.
-    ``names`` as for ``pre_norm``; a layer without a feed-forward is its first half only."""
+    ``residual_factor`` multiplies both norms' outputs.  ``names`` as for ``pre_norm``; a layer without a feed-forward is its
+    first half only."""
 
     graph_safe = True
 
     def __init__(
         self, *, mixer: Mapping[str, Any], feed_forward: Mapping[str, Any] | None, mixer_norm: Mapping[str, Any],
-        ffn_norm: Mapping[str, Any] | None = None, names: Mapping[str, str] | None = None,
+        ffn_norm: Mapping[str, Any] | None = None, names: Mapping[str, str] | None = None, residual_factor: float = 1.0,
     ) -> None:
+        self.residual_factor = float(residual_factor)
         self.names = {**_DEFAULT_NAMES, **(names or {})}
         self.mixer = MIXERS.build(mixer)
         self.mixer_norm = NORMS.build(mixer_norm)
@@ -130,13 +132,13 @@ class OutputNormBlock(Block):
             x = M.norm_accumulate_round(None, None, 0.0, resid, act) if rounds else resid
         out = self.mixer.forward(x, ctx, cache)
         weight, eps = self.mixer_norm.fusable()
-        x = M.norm_accumulate_round(out, weight, eps, resid, act if rounds else None)
+        x = M.norm_accumulate_round(out, weight, eps, resid, act if rounds else None, self.residual_factor)
         if self.feed_forward is not None:
             # a feed-forward that can hand over its experts' rows unsummed does: the norm's kernel forms the sum
             pieces = {"pieces": True} if getattr(self.feed_forward, "returns_pieces", False) else {}
             out = self.feed_forward.forward(x if rounds else resid, ctx, **pieces)
             weight, eps = self.ffn_norm.fusable()
-            x = M.norm_accumulate_round(out, weight, eps, resid, act if rounds else None)
+            x = M.norm_accumulate_round(out, weight, eps, resid, act if rounds else None, self.residual_factor)
         if rounds:
             stream.rounded = x
 

@@ -161,7 +161,8 @@ class LatentAttention(Mixer):
     is one key part shared by all heads, rotated by the position (``position``: a rotary encoding over the first columns of the
     ``rot_dim``; ``None``: no rotation).  Per
     head the plain key is ``W_uk c`` and the value ``W_uv c``; ``S = scale * (q_plain . k_plain + q_rot . k_rot)``; a window as in
-    ``gated_attention``; softmax; the heads side by side are multiplied element by element with ``sigmoid(W_g x)``; then ``W_o``.
+    ``gated_attention``; softmax, with ``sink`` over one more term ``exp(sink_h)`` per head that belongs to no key; the heads side by
+    side are multiplied with ``sigmoid(W_g x)``, element by element (``gate="element"``) or one number per head (``"head"``); then ``W_o``.
 
     Only ``c`` and the rotated key part are kept per token (one row of ``kv_rank + rot_dim`` columns).  The products with
     ``W_uk`` and ``W_uv`` are moved to the query's side: ``q_plain . (W_uk c) = (W_uk^T q_plain) . c`` and
@@ -169,15 +170,18 @@ class LatentAttention(Mixer):
     are also the values.  ``shares_kv``: the layer has no ``W_dkv`` and reads the rows another layer wrote.  ``keep_window``:
     how far back the kept rows are read by this layer or by any layer that borrows them (``None``: everything).
 
-    Tensors: ``dq``, ``dkv``, ``g`` (one stacked product), ``dq.norm``, ``dkv.norm``, ``uq``, ``uk``, ``uv``, ``o``."""
+    Tensors: ``dq``, ``dkv``, ``g`` (one stacked product), ``dq.norm``, ``dkv.norm``, ``uq``, ``uk``, ``uv``, ``sink``, ``o``."""
 
     graph_safe = True
 
     def __init__(self, *, hidden_size: int, num_heads: int, head_dim: int, rot_dim: int, value_dim: int, kv_rank: int, q_rank: int,
                  eps: float, position: Mapping[str, Any] | None = None, scale: float | None = None, window: int | None = None,
-                 shares_kv: bool = False, keep_window: int | None = None) -> None:
+                 shares_kv: bool = False, keep_window: int | None = None, sink: bool = False, gate: str = "element") -> None:
         if min(hidden_size, num_heads, head_dim, value_dim, kv_rank, q_rank) <= 0 or rot_dim < 0:
             raise ValueError("latent attention sizes must be positive")
+        if gate not in ("element", "head"):
+            raise ValueError(f"latent attention's gate is per element or per head, got {gate!r}")
+        self.has_sink, self.gate = bool(sink), gate
         self.hidden_size, self.num_heads, self.head_dim, self.rot_dim = hidden_size, num_heads, head_dim, rot_dim
         self.value_dim, self.kv_rank, self.q_rank, self.eps = value_dim, kv_rank, q_rank, float(eps)
         self.scale = 1.0 / math.sqrt(head_dim + rot_dim) if scale is None else float(scale)
@@ -195,8 +199,10 @@ class LatentAttention(Mixer):
             "dkv": TensorSpec((self.kv_rank + self.rot_dim, h)),
             "dkv.norm": TensorSpec((self.kv_rank,), init="one_plus_normal", std=0.05),
             "uk": TensorSpec((H * self.head_dim, self.kv_rank)), "uv": TensorSpec((H * self.value_dim, self.kv_rank)),
-            "g": TensorSpec((H * self.value_dim, h)), "o": TensorSpec((h, H * self.value_dim)),
+            "g": TensorSpec((H if self.gate == "head" else H * self.value_dim, h)), "o": TensorSpec((h, H * self.value_dim)),
         }
+        if self.has_sink:
+            specs["sink"] = TensorSpec((H,), init="normal", std=0.5)
         if self.shares_kv:
             del specs["dkv"], specs["dkv.norm"]
         return specs
@@ -213,6 +219,7 @@ class LatentAttention(Mixer):
         self.uk = runtime.place_matrix(tensors["uk"]).view(H, self.head_dim, self.kv_rank).transpose(1, 2).contiguous()
         self.uv = runtime.place_matrix(tensors["uv"]).view(H, self.value_dim, self.kv_rank)
         self.o_proj = Projection([tensors["o"]], None, runtime)
+        self.sink = runtime.place_vector_f32(tensors["sink"]) if self.has_sink else None
         if self.position is not None:
             self.position.load({}, runtime)
 
@@ -225,12 +232,13 @@ class LatentAttention(Mixer):
         proj = self.in_proj(x)
         table = ctx.block_table(cache.group)
         pool = cache.tensors["latent"]
-        inv_freq, rot_dims = self.position.rotary_parameters() if self.position is not None else (None, 0)
+        inv_freq, rot_dims, interleaved, factor = self.position.rotary_layout() if self.position is not None else (None, 0, False, 1.0)
         own = not self.shares_kv
         cq = M.latent_prepare(
             proj, q_offset=0, q_rank=self.q_rank, q_weight=self.q_weight, eps=self.eps, positions=ctx.positions,
             token_entry=ctx.token_entry, kv_offset=self.q_rank, kv_rank=self.kv_rank if own else 0, kv_weight=self.kv_weight,
             rot=self.rot_dim, rot_dims=rot_dims, inv_freq=inv_freq, block_table=table, page_size=cache.page_size, pool=pool,
+            interleaved=interleaved, rot_factor=factor,
         )
         q = self.uq_proj(cq)
         n, H, row = q.shape[0], self.num_heads, self.kv_rank + self.rot_dim
@@ -240,11 +248,12 @@ class LatentAttention(Mixer):
                          out=absorbed, out_batch_stride=row)
         if self.rot_dim:
             M.rope_slice(q, absorbed, heads=H, src_head=q_head, src_offset=self.head_dim, dst_head=row, dst_offset=self.kv_rank,
-                         rot=self.rot_dim, rot_dims=rot_dims, inv_freq=inv_freq, positions=ctx.positions)
+                         rot=self.rot_dim, rot_dims=rot_dims, inv_freq=inv_freq, positions=ctx.positions, interleaved=interleaved,
+                         rot_factor=factor)
         mixed = attention_latent.latent_attention(absorbed.view(n, H, row), pool, ctx, table, value_dim=self.kv_rank, scale=self.scale,
-                                                  window=self.window or 0)
+                                                  window=self.window or 0, sink=self.sink)
         out = G.batched_linear(mixed.view(n, H * self.kv_rank), self.uv, batch=H, k=self.kv_rank, n_out=self.value_dim,
                                a_batch_stride=self.kv_rank)
         gate_offset = self.q_rank + (self.kv_rank + self.rot_dim if own else 0)
-        gated = M.sigmoid_gate(out, proj, gate_offset=gate_offset, group=1)
+        gated = M.sigmoid_gate(out, proj, gate_offset=gate_offset, group=1 if self.gate == "element" else self.value_dim)
         return self.o_proj(gated, torch.float32)

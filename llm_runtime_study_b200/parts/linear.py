@@ -73,26 +73,26 @@ class Projection:
             return x.values, {"row_scale": x.scale}
         return x.normalised(), {}
 
-    def swiglu(self, x: "torch.Tensor | WeightedRows") -> torch.Tensor:
+    def swiglu(self, x: "torch.Tensor | WeightedRows", act: str = "silu") -> torch.Tensor:
         """For a projection whose rows are gate and up features interleaved in blocks of
-        eight: ``silu(gate(x)) * up(x)`` in the activation type.  Our bfloat16 kernels apply
+        eight: ``silu(gate(x)) * up(x)`` (``act``: or another gate) in the activation type.  Our bfloat16 kernels apply
         the activation in their epilogue, so the ``[tokens, 2 I]`` intermediate is never
         written; the other paths run the projection and then the interleaved SiLU kernel."""
 
         x, norm = self._unweighted(x)
         if norm:
-            return gemm_bf16.linear_skinny(x, self.weight, self.bias, torch.bfloat16, swiglu=True, **norm)
+            return gemm_bf16.linear_skinny(x, self.weight, self.bias, torch.bfloat16, swiglu=act, **norm)
         if self.runtime.dtype == torch.bfloat16 and self.in_features % 8 == 0 and x.is_contiguous():
             m = x.shape[0]
             if m <= gemm_bf16.SKINNY_M:
                 if self.GEMM_BACKEND == "tcgen05" and gemm_bf16.few_rows_kernel(m, self.out_features, self.in_features) == "splitk":
-                    return gemm_bf16.linear(x, self.weight, self.bias, torch.bfloat16, swiglu=True, kernel="splitk")
-                return gemm_bf16.linear_skinny(x, self.weight, self.bias, torch.bfloat16, swiglu=True)
+                    return gemm_bf16.linear(x, self.weight, self.bias, torch.bfloat16, swiglu=act, kernel="splitk")
+                return gemm_bf16.linear_skinny(x, self.weight, self.bias, torch.bfloat16, swiglu=act)
             if self.GEMM_BACKEND == "tcgen05" and m >= self.TCGEN05_MIN_ROWS:
-                return gemm_bf16.linear(x, self.weight, self.bias, torch.bfloat16, swiglu=True)
+                return gemm_bf16.linear(x, self.weight, self.bias, torch.bfloat16, swiglu=act)
             if self.GEMM_BACKEND == "tcgen05" and self.MID_ROWS == "splitk":
-                return gemm_bf16.linear(x, self.weight, self.bias, torch.bfloat16, swiglu=True, kernel="splitk")
-        return F.silu_mul_interleaved(self(x))
+                return gemm_bf16.linear(x, self.weight, self.bias, torch.bfloat16, swiglu=act, kernel="splitk")
+        return F.silu_mul_interleaved(self(x), act)
 
     def __call__(self, x: "torch.Tensor | WeightedRows", out_dtype: torch.dtype | None = None, *,
                  add_to: torch.Tensor | None = None, next_norm: Any = None) -> "torch.Tensor | WeightedRows | None":

@@ -155,6 +155,118 @@ class GatedDeltaRule(Mixer):
         return self.o_proj(gated, torch.float32)
 
 
+@MIXERS.register("gated_linear_attention")
+class GatedLinearAttention(Mixer):
+    """Linear attention with one decay per key channel (the gated linear attention of Yang et al.): ``q = W_q x * dim^(-1/2)``,
+    ``k = W_k x`` (``heads x dim``), ``v = W_v x`` (``heads x vdim``), ``alpha = sigmoid(W_a2 (W_a1 x) + a2.b)^(1 / tau)`` (``heads x
+    dim``); per head ``S <- diag(alpha) S + k v^T``, ``o = S^T q``.  Each head's ``o`` is RMS-normed with one weight of ``vdim`` numbers
+    for all heads (``norm``), the heads side by side are multiplied with ``silu(W_g x)``, then ``W_o``.  The state
+    ``[heads, dim, vdim]`` is float32, starts at zero and lives in the request's slot.  Tensors: ``q``, ``k``, ``v``, ``g``, ``a1`` (one
+    stacked product), ``a2``, ``a2.b``, ``norm``, ``o``."""
+
+    graph_safe = True
+
+    def __init__(self, *, hidden_size: int, num_heads: int, head_dim: int, value_dim: int, decay_rank: int, tau: float, eps: float) -> None:
+        if min(hidden_size, num_heads, head_dim, value_dim, decay_rank) <= 0 or head_dim > 256 or tau <= 0:
+            raise ValueError("gated linear attention's sizes and tau must be positive, the key size at most 256")
+        self.hidden_size, self.num_heads, self.head_dim, self.value_dim = hidden_size, num_heads, head_dim, value_dim
+        self.decay_rank, self.tau, self.eps = decay_rank, float(tau), float(eps)
+
+    def tensor_specs(self) -> dict[str, TensorSpec]:
+        qk, vw, h = self.num_heads * self.head_dim, self.num_heads * self.value_dim, self.hidden_size
+        return {
+            "q": TensorSpec((qk, h)), "k": TensorSpec((qk, h)), "v": TensorSpec((vw, h)), "g": TensorSpec((vw, h)),
+            "a1": TensorSpec((self.decay_rank, h)), "a2": TensorSpec((qk, self.decay_rank)),
+            "a2.b": TensorSpec((qk,), init="normal", std=0.5),
+            "norm": TensorSpec((self.value_dim,), init="one_plus_normal", std=0.05), "o": TensorSpec((h, vw)),
+        }
+
+    def load(self, tensors: Mapping[str, torch.Tensor], runtime: Runtime) -> None:
+        self.runtime = runtime
+        self.in_proj = _padded([tensors[n] for n in ("q", "k", "v", "g", "a1")], runtime)
+        # the second half of the low-rank map is applied inside the kernel that forms the decays, which reads it transposed
+        self.a_up = runtime.place_matrix(tensors["a2"]).t().contiguous()
+        self.a_bias = runtime.place_vector_f32(tensors["a2.b"])
+        self.norm_weight = runtime.place_vector_f32(tensors["norm"])
+        self.o_proj = Projection([tensors["o"]], None, runtime)
+
+    def cache_requirement(self) -> FixedState:
+        return FixedState((self.num_heads, self.head_dim, self.value_dim), torch.float32)
+
+    def forward(self, x: torch.Tensor, ctx: Any, cache: Any) -> torch.Tensor:
+        proj = self.in_proj(x)
+        qk, vw = self.num_heads * self.head_dim, self.num_heads * self.value_dim
+        alpha = S.channel_decay(proj, self.a_up, self.a_bias, offset=2 * (qk + vw), tau=self.tau)
+        out = S.linear_scan(
+            proj[:, :qk], proj[:, qk : 2 * qk], proj[:, 2 * qk : 2 * qk + vw], heads=self.num_heads, qk_heads=self.num_heads,
+            dim=self.head_dim, vdim=self.value_dim, state=cache.state, q_start=ctx.q_start, slots=ctx.slots, gate=alpha,
+            q_scale=self.head_dim ** -0.5, fixed_order=self.runtime.dtype == torch.float32,
+        )
+        gated = S.group_norm_gate(out, self.norm_weight, self.eps, proj, gate_offset=2 * qk + vw, act="silu", out_dtype=self.runtime.dtype)
+        return self.o_proj(gated, torch.float32)
+
+
+@MIXERS.register("matrix_memory")
+class MatrixMemory(Mixer):
+    """The matrix memory of xLSTM (mLSTM): ``q = W_q x * dim^(-1/2)``, ``k = W_k x`` (``heads x dim``), ``v = W_v x`` (``heads x
+    vdim``); per head ``i = cap tanh((W_i x + i.b) / cap)`` and ``f = ln sigmoid(cap tanh((W_f x + f.b) / cap))`` with ``cap`` =
+    ``gate_cap``.  With a running maximum ``m_t = max(f + m_(t-1), i)`` from 0: ``S <- exp(f + m_(t-1) - m_t) S + exp(i - m_t) k v^T``,
+    ``n`` likewise with ``k`` alone, ``o = S^T q / (max(|n . q|, exp(-m_t)) + 1e-6)``.  Each head's ``o`` is divided by its root mean
+    square (``eps``); the heads side by side times ``norm`` (all heads' size) and ``sigmoid(W_g x)``, then ``W_o``.
+
+    Per request, float32 from zero: ``S`` ``[heads, dim, vdim]``, ``n`` ``[heads, dim]``, ``m`` ``[heads]``.  Tensors: ``q``, ``k``, ``v``,
+    ``g``, ``i``, ``f`` (one stacked product), ``i.b``, ``f.b``, ``norm``, ``o``."""
+
+    graph_safe = True
+    NORMALISER_EPS = 1e-6
+
+    def __init__(self, *, hidden_size: int, num_heads: int, head_dim: int, value_dim: int, gate_cap: float, eps: float) -> None:
+        if min(hidden_size, num_heads, head_dim, value_dim) <= 0 or head_dim > 256 or gate_cap <= 0:
+            raise ValueError("a matrix memory's sizes and gate cap must be positive, the key size at most 256")
+        self.hidden_size, self.num_heads, self.head_dim, self.value_dim = hidden_size, num_heads, head_dim, value_dim
+        self.gate_cap, self.eps = float(gate_cap), float(eps)
+
+    def tensor_specs(self) -> dict[str, TensorSpec]:
+        qk, vw, h, H = self.num_heads * self.head_dim, self.num_heads * self.value_dim, self.hidden_size, self.num_heads
+        return {
+            "q": TensorSpec((qk, h)), "k": TensorSpec((qk, h)), "v": TensorSpec((vw, h)), "g": TensorSpec((vw, h)),
+            "i": TensorSpec((H, h)), "i.b": TensorSpec((H,), init="normal", std=0.5),
+            "f": TensorSpec((H, h)), "f.b": TensorSpec((H,), init="one_plus_normal", std=0.5),
+            "norm": TensorSpec((vw,), init="one_plus_normal", std=0.05), "o": TensorSpec((h, vw)),
+        }
+
+    def load(self, tensors: Mapping[str, torch.Tensor], runtime: Runtime) -> None:
+        self.runtime = runtime
+        self.in_proj = _padded([tensors[n] for n in ("q", "k", "v", "g", "i", "f")], runtime)
+        self.i_bias, self.f_bias = runtime.place_vector_f32(tensors["i.b"]), runtime.place_vector_f32(tensors["f.b"])
+        self.norm_weight = runtime.place_vector_f32(tensors["norm"])
+        self.o_proj = Projection([tensors["o"]], None, runtime)
+
+    def cache_requirement(self):
+        return (
+            FixedState((self.num_heads, self.head_dim, self.value_dim), torch.float32, name="state"),
+            FixedState((self.num_heads, self.head_dim), torch.float32, name="normaliser"),
+            FixedState((self.num_heads,), torch.float32, name="maximum"),
+        )
+
+    def forward(self, x: torch.Tensor, ctx: Any, cache: Any) -> torch.Tensor:
+        proj = self.in_proj(x)                      # [N, q | k | v | g | i | f]
+        H, qk, vw = self.num_heads, self.num_heads * self.head_dim, self.num_heads * self.value_dim
+        i_offset = 2 * (qk + vw)
+        decay, gain, floor = S.memory_gates(
+            proj, heads=H, i_offset=i_offset, f_offset=i_offset + H, i_bias=self.i_bias, f_bias=self.f_bias, cap=self.gate_cap,
+            m_state=cache.states["maximum"], q_start=ctx.q_start, slots=ctx.slots,
+        )
+        out, den = S.linear_scan_row_gates(
+            proj[:, :qk], proj[:, qk : 2 * qk], proj[:, 2 * qk : 2 * qk + vw], heads=H, dim=self.head_dim, vdim=self.value_dim,
+            decay=decay, gain=gain, state=cache.states["state"], norm_state=cache.states["normaliser"], q_start=ctx.q_start,
+            slots=ctx.slots, q_scale=self.head_dim ** -0.5, fixed_order=self.runtime.dtype == torch.float32,
+        )
+        gated = S.group_norm_gate(out, self.norm_weight, self.eps, proj, gate_offset=2 * qk + vw, group=self.value_dim,
+                                  divisor=(den, floor, self.NORMALISER_EPS), out_dtype=self.runtime.dtype)
+        return self.o_proj(gated, torch.float32)
+
+
 @MIXERS.register("parallel")
 class ParallelMixers(Mixer):
     """Several mixers side by side on the same rows.  Each branch's output is RMS-normalised over the model

@@ -1,8 +1,8 @@
-"""Gated feed-forward (SwiGLU)."""
+"""Dense feed-forwards."""
 
 from __future__ import annotations
 
-from typing import Any, Mapping
+from typing import Any, Mapping, Sequence
 
 import torch
 
@@ -14,29 +14,32 @@ from .linear import Projection
 
 
 @FEED_FORWARDS.register("swiglu")
-class SwiGLU(FeedForward):
-    """``down(silu(gate(x)) * up(x))`` without biases (mini_llm/nn/mlp.py:80-87).
-    gate and up are one stacked product; the activation and the product with
-    ``up`` are computed in float32 and rounded once."""
+class GatedMLP(FeedForward):
+    """``down(act(gate(x)) * up(x))`` without biases, ``act`` being SiLU (mini_llm/nn/mlp.py:80-87) or the tanh
+    form of gelu (``act="gelu_tanh"``).  gate and up are one stacked product; the activation and the product with
+    ``up`` are computed in float32 and rounded once.  ``names``: the checkpoint's names of gate, up and down."""
 
     graph_safe = True
 
-    def __init__(self, *, hidden_size: int, intermediate_size: int) -> None:
+    def __init__(self, *, hidden_size: int, intermediate_size: int, act: str = "silu",
+                 names: Sequence[str] = ("gate_proj.weight", "up_proj.weight", "down_proj.weight")) -> None:
         if hidden_size <= 0 or intermediate_size <= 0:
             raise ValueError("swiglu sizes must be positive")
-        self.hidden_size, self.intermediate_size = hidden_size, intermediate_size
+        if act not in F.GATE_ACTS or len(names) != 3:
+            raise ValueError(f"a gated feed-forward takes one of {sorted(F.GATE_ACTS)} and three names, got {act!r}, {names}")
+        self.hidden_size, self.intermediate_size, self.act, self.names = hidden_size, intermediate_size, act, tuple(names)
 
     def tensor_specs(self) -> dict[str, TensorSpec]:
         h, i = self.hidden_size, self.intermediate_size
         return {
-            "gate_proj.weight": TensorSpec((i, h)),
-            "up_proj.weight": TensorSpec((i, h)),
-            "down_proj.weight": TensorSpec((h, i)),
+            self.names[0]: TensorSpec((i, h)),
+            self.names[1]: TensorSpec((i, h)),
+            self.names[2]: TensorSpec((h, i)),
         }
 
     def load(self, tensors: Mapping[str, torch.Tensor], runtime: Runtime) -> None:
         self.runtime = runtime
-        gate, up = runtime.place_matrix(tensors["gate_proj.weight"]), runtime.place_matrix(tensors["up_proj.weight"])
+        gate, up = runtime.place_matrix(tensors[self.names[0]]), runtime.place_matrix(tensors[self.names[1]])
         # When the width allows, gate and up rows are interleaved in blocks of eight
         # ([g0..g7, u0..u7, g8..g15, ...]): a projection kernel then holds matching gate and
         # up features in one tile and can apply SiLU * up before it writes anything.
@@ -49,14 +52,17 @@ class SwiGLU(FeedForward):
             del stacked
         else:
             self.gate_up_proj = Projection([gate, up], None, runtime)
-        self.down_proj = Projection([tensors["down_proj.weight"]], None, runtime)
+        self.down_proj = Projection([tensors[self.names[2]]], None, runtime)
 
     adds_to_residual = True
     fuses_norms = True
 
     def forward(self, x: Any, ctx: Any, residual: torch.Tensor | None = None, next_norm: Any = None):
-        hidden = self.gate_up_proj.swiglu(x) if self.interleaved else F.silu_mul(self.gate_up_proj(x))
+        hidden = self.gate_up_proj.swiglu(x, self.act) if self.interleaved else F.silu_mul(self.gate_up_proj(x), self.act)
         return self.down_proj(hidden, torch.float32, add_to=residual, next_norm=next_norm)
+
+
+FEED_FORWARDS.register("gated_mlp", GatedMLP)
 
 
 @FEED_FORWARDS.register("limited_glu")
