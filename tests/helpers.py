@@ -535,3 +535,81 @@ def make_tafisun_dir(path: Path, config: dict, seed: int, *, torch_dtype: str = 
     (path / "config.json").write_text(json.dumps(config, indent=1), encoding="utf-8")
     write_file(path / "model.safetensors", state)
     return path, state
+
+
+# ----------------------------------------------------------------- Fumolorn
+# A: sizes that are no multiples of 16, values wider and narrower than keys, a rotation stretched so that some pairs keep
+# their frequency, some are divided and some lie between, a single head of matrix memory, a layer without a feed-forward, a
+# bigram table of 13 rows (many pairs collide) with multipliers that overflow 32 bits, caps low enough to bite.
+FUMOLORN_A = {
+    "architecture": "Fumolorn", "vocab": 211, "width": 64, "norm": {"eps": 1e-5}, "residual_mult": 0.6, "logit_softcap": 4.0,
+    "embedding": {"scale": 3.5, "bigram": {"buckets": 13, "mul_prev": 40_000_003, "mul_cur": 11}},
+    "layers": [
+        {"type": "mlstm", "mixer": {"heads": 1, "dim": 24, "vdim": 40, "gate_cap": 5.0}, "mlp": {"kind": "dense", "ff": 72}},
+        {"type": "latent_attention", "mixer": {"heads": 3, "dim": 16, "rot_dim": 12, "vdim": 24, "kv_rank": 40, "q_rank": 48, "scale": 0.35,
+                                               "rot": {"base": 500.0, "dims": 12, "scaling": {"factor": 4.0, "original": 64, "fast": 8.0, "slow": 1.0}}},
+         "mlp": None},
+        {"type": "gla", "mixer": {"heads": 3, "dim": 12, "vdim": 20, "tau": 8.0}, "mlp": {"kind": "dense", "ff": 50}},
+        {"type": "mlstm", "mixer": {"heads": 5, "dim": 16, "vdim": 8, "gate_cap": 15.0}, "mlp": {"kind": "dense", "ff": 40}},
+        {"type": "latent_attention", "mixer": {"heads": 2, "dim": 8, "rot_dim": 4, "vdim": 12, "kv_rank": 24, "q_rank": 20, "scale": 0.5,
+                                               "rot": {"base": 100.0, "dims": 4}},
+         "mlp": {"kind": "dense", "ff": 56}},
+    ],
+}
+# B: every factor 1 (embedding scale, residual multiplier, tau), no cap on the logits, no bigram table, one head of attention
+# without a rotation's scaling, a width that no vector divides.
+FUMOLORN_B = {
+    "architecture": "Fumolorn", "vocab": 131, "width": 50, "norm": {"eps": 1e-6}, "residual_mult": 1.0, "logit_softcap": None,
+    "embedding": {"scale": 1.0, "bigram": None},
+    "layers": [
+        {"type": "gla", "mixer": {"heads": 1, "dim": 40, "vdim": 7, "tau": 1.0}, "mlp": None},
+        {"type": "latent_attention", "mixer": {"heads": 1, "dim": 24, "rot_dim": 16, "vdim": 40, "kv_rank": 20, "q_rank": 12, "scale": 0.16,
+                                               "rot": {"base": 10000.0, "dims": 16, "scaling": None}}, "mlp": {"kind": "dense", "ff": 33}},
+        {"type": "mlstm", "mixer": {"heads": 2, "dim": 9, "vdim": 33, "gate_cap": 1.5}, "mlp": {"kind": "dense", "ff": 64}},
+    ],
+}
+# C: sizes in steps of 16 throughout, which is what the tensor-core kernels of the bfloat16 run type take.
+FUMOLORN_C = {
+    "architecture": "Fumolorn", "vocab": 152, "width": 128, "norm": {"eps": 1e-6}, "residual_mult": 0.5, "logit_softcap": 20.0,
+    "embedding": {"scale": 11.0, "bigram": {"buckets": 97, "mul_prev": 29, "mul_cur": 5}},
+    "layers": [
+        {"type": "latent_attention", "mixer": {"heads": 5, "dim": 16, "rot_dim": 16, "vdim": 32, "kv_rank": 32, "q_rank": 48, "scale": 0.25,
+                                               "rot": {"base": 5000.0, "dims": 16, "scaling": {"factor": 16.0, "original": 128, "fast": 16.0, "slow": 2.0}}},
+         "mlp": {"kind": "dense", "ff": 256}},
+        {"type": "gla", "mixer": {"heads": 4, "dim": 64, "vdim": 32, "tau": 16.0}, "mlp": {"kind": "dense", "ff": 192}},
+        {"type": "mlstm", "mixer": {"heads": 2, "dim": 32, "vdim": 64, "gate_cap": 10.0}, "mlp": {"kind": "dense", "ff": 256}},
+        {"type": "latent_attention", "mixer": {"heads": 3, "dim": 64, "rot_dim": 16, "vdim": 16, "kv_rank": 64, "q_rank": 32, "scale": 0.12,
+                                               "rot": {"base": 5000.0, "dims": 16, "scaling": {"factor": 2.0, "original": 4096, "fast": 32.0, "slow": 1.0}}},
+         "mlp": {"kind": "dense", "ff": 256}},
+    ],
+}
+FUMOLORN = {"A": (FUMOLORN_A, 51, 4), "B": (FUMOLORN_B, 52, 16), "C": (FUMOLORN_C, 53, 16)}   # config, seed, page size
+
+
+def make_fumolorn_dir(path: Path, config: dict, seed: int, *, torch_dtype: str = "float32", gain: float = 6.0, ranks: dict | None = None):
+    """Write a Fumolorn model folder with random weights; return (path, {name: CPU tensor as stored}).  The matrices are
+    drawn ``gain`` times larger than the framework's default, so that gates and scores are not all alike."""
+
+    from llm_runtime_study_b200.config import FumolornConfig
+    from llm_runtime_study_b200.models.description import tensor_schema
+    from llm_runtime_study_b200.models.fumolorn import describe_fumolorn
+    from llm_runtime_study_b200.weights.random_init import random_state
+    from llm_runtime_study_b200.weights.safetensors_io import write_file
+
+    schema = tensor_schema(describe_fumolorn(FumolornConfig.from_dict(config), ranks))
+    dtype = {"float32": torch.float32, "bfloat16": torch.bfloat16}[torch_dtype]
+    state = random_state(schema, seed, dtype=torch.float32, include_optional=False)
+    for name, tensor in state.items():
+        if name in ("embed", "bigram"):
+            tensor *= 40.0
+        elif name.endswith(".f.b"):
+            tensor += 2.0                # most of what a matrix memory holds outlives a step
+        elif name.endswith(".a2.b"):
+            tensor += 2.0
+        elif tensor.dim() == 2:
+            tensor *= gain
+    state = {name: tensor.to(dtype) for name, tensor in state.items()}
+    path.mkdir(parents=True, exist_ok=True)
+    (path / "config.json").write_text(json.dumps(config, indent=1), encoding="utf-8")
+    write_file(path / "model.safetensors", state)
+    return path, state
