@@ -1312,6 +1312,192 @@ def _tafisun_kernels(peak, timed) -> dict:
     return out
 
 
+# ------------------------------------------------------------------------------ Fumolorn beside Ropulix, Sorulix and Qwen3
+def _fumolorn_config(width, ff, heads, kv_heads, d, pairs, vocab) -> dict:
+    """A gated linear attention layer, a latent attention layer, a matrix memory layer and a latent attention layer in turn; the
+    recurrences keep ``heads`` states of ``d x d`` and the latent rows are as wide as in the Ropulix configuration."""
+
+    latent = {"heads": heads, "dim": d, "rot_dim": d // 2, "vdim": d, "kv_rank": 4 * d, "q_rank": width // 2, "scale": (d + d // 2) ** -0.5,
+              "rot": {"base": 50000.0, "dims": d // 2, "scaling": {"factor": 8.0, "original": 1024, "fast": 32.0, "slow": 1.0}}}
+    mlp = {"kind": "dense", "ff": ff}
+    layers = []
+    for _ in range(pairs):
+        layers += [
+            {"type": "gla", "mixer": {"heads": heads, "dim": d, "vdim": d, "tau": 16.0}, "mlp": mlp},
+            {"type": "latent_attention", "mixer": latent, "mlp": mlp},
+            {"type": "mlstm", "mixer": {"heads": heads, "dim": d, "vdim": d, "gate_cap": 15.0}, "mlp": mlp},
+            {"type": "latent_attention", "mixer": latent, "mlp": mlp},
+        ]
+    return {"architecture": "Fumolorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "torch_dtype": "bfloat16",
+            "residual_mult": 0.5, "logit_softcap": 30.0, "layers": layers[: 2 * pairs],
+            "embedding": {"scale": width ** 0.5, "bigram": {"buckets": 65521, "mul_prev": 131, "mul_cur": 17}}}
+
+
+def run_fumolorn(args) -> dict:
+    """Prefill and decode of Fumolorn at layer sizes of real models (random weights), beside Ropulix (the other design with latent
+    attention and norms on the sublayers' outputs), Sorulix (the other design with matrix states per request) and Qwen3 at equal
+    width, heads, head size and depth, through the same engine; then the new kernels alone against the bytes or flops they must
+    move, each beside the like kernel of an existing path."""
+
+    peak, timed, measure = _engine_measurer(args)
+    results = {}
+    for name in (() if args.only == "kernels" else args.size.split(",") if args.size else SORULIX_SIZES):
+        shape = SORULIX_SIZES[name]
+        results[name] = {"shape": dict(zip(("width", "ff", "heads", "kv_heads", "head_dim", "layer_pairs", "vocab"), shape)),
+                         "fumolorn": measure(_fumolorn_config(*shape), shape[-1])}
+        if args.only not in ("prefill", "decode"):
+            results[name]["ropulix_equal_size"] = measure(_ropulix_config(*shape), shape[-1])
+            results[name]["sorulix_equal_size"] = measure(_sorulix_config(*shape), shape[-1])
+            results[name]["qwen3_equal_size"] = measure(_qwen3_like(*shape), shape[-1])
+    kernels = _fumolorn_kernels(peak, timed) if args.only in ("all", "kernels") else {}
+    return {"workload": "fumolorn", "context": CONTEXT, "steps": args.steps, "warmup": max(args.warmup, 3), "dtype": "bfloat16",
+            "data": "synthetic token ids, seeded random weights", "peaks": peak, "models": results, "kernels": kernels}
+
+
+def _fumolorn_kernels(peak, timed) -> dict:
+    """Each new kernel alone at the 4k shape (width 4096, 32 heads of 128), replayed from a CUDA graph, beside the kernel of an
+    existing path that does the like work; fractions are of the measured copy bandwidth for the bytes a kernel must move, or of
+    the measured bf16 rate for its products."""
+
+    import torch
+    from types import SimpleNamespace
+
+    from llm_runtime_study_b200.ops import attention_latent, gemm_bf16
+    from llm_runtime_study_b200.ops import functional as F
+    from llm_runtime_study_b200.ops import mixer_steps as M
+    from llm_runtime_study_b200.ops import sequence_state as S
+
+    dev = "cuda:0"
+    width, heads, d, ff, page = 4096, 32, 128, 12288, PAGE_SIZE
+    vw = heads * d
+    out = {}
+    cold = timed
+
+    def timed(fn, repeat):
+        fn()
+        fn()
+        torch.cuda.synchronize()
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph):
+            fn()
+        graph.replay()
+        return cold(graph.replay, repeat)
+
+    def beside(new, old, moved_new=None, moved_old=None, flops=None):
+        """Microseconds of the new kernel and of the like one, and their fractions of the measured rates."""
+
+        t_new, t_old = timed(new, 20), timed(old, 20)
+        row = {"us": round(t_new * 1e3, 1), "like_us": round(t_old * 1e3, 1)}
+        if moved_new is not None:
+            row["of_measured_copy"] = [round(m / t / 1e6 / peak["hbm_gbs"], 3) for m, t in ((moved_new, t_new), (moved_old or moved_new, t_old))]
+        if flops is not None:
+            row["of_measured_bf16_burst"] = [round(flops / t / 1e9 / peak["bf16_tflops"], 4) for t in (t_new, t_old)]
+        return row
+
+    bf = lambda *shape: (0.05 * torch.randn(*shape, device=dev)).bfloat16()
+    f32 = lambda *shape: torch.randn(*shape, device=dev)
+    ints = lambda values: torch.tensor(values, dtype=torch.int32, device=dev)
+    # latent attention with sinks beside the same without (both see every key)
+    rank, rot = 4 * d, d // 2
+    sink = f32(heads)
+    for seqs, length, new in ((1, 2048, 2048), (8, 2048, 1), (32, 2048, 1)):
+        lengths, q_lens = [length] * seqs, [new] * seqs
+        table = torch.arange(seqs * (length // page), dtype=torch.int32).view(seqs, -1).to(dev)
+        pool, q = bf(seqs * (length // page), page, rank + rot), bf(seqs * new, heads, rank + rot)
+        positions = ints([p for m, k in zip(lengths, q_lens) for p in range(m - k, m)])
+        entry = ints([i for i, k in enumerate(q_lens) for _ in range(k)])
+        ctx = SimpleNamespace(positions=positions, token_entry=entry, all_decode=new == 1, num_entries=seqs, q_lens=q_lens, kv_lens=lengths,
+                              max_kv_len=length)
+        run = lambda s: attention_latent.latent_attention(q, pool, ctx, table, value_dim=rank, scale=0.07, sink=s)
+        flops = 2.0 * heads * sum(p + 1 for p in positions.tolist()) * (2 * rank + rot)
+        out[f"latent_attention_{seqs}x{length}_new_{new}"] = beside(
+            lambda: run(sink), lambda: run(None), None if new > 1 else seqs * length * (rank + rot) * 2, flops=flops)
+    # the scans: row gates and channel decays beside the constant decay and the gated delta rule
+    for n, entries in ((2048, 1), (8, 8), (64, 64)):
+        q, k, v = bf(n, vw), bf(n, vw), bf(n, vw)
+        state, norm_state = torch.zeros(entries + 1, heads, d, d, device=dev), torch.zeros(entries + 1, heads, d, device=dev)
+        q_start, slots = ints(list(range(0, n + 1, n // entries))), ints(list(range(entries)))
+        decay, gain, const = torch.rand(n, heads, device=dev), torch.rand(n, heads, device=dev), torch.full((heads,), 0.97, device=dev)
+        gate, beta = 0.9 + 0.1 * torch.rand(n, vw, device=dev), torch.rand(n, heads, device=dev)
+        moved = 2.0 * entries * heads * d * d * 4 + n * vw * 10
+        sizes = dict(heads=heads, qk_heads=heads, dim=d, vdim=d, state=state, q_start=q_start, slots=slots)
+        out[f"scan_row_gates_{n}_tokens_{entries}_requests"] = beside(
+            lambda: S.linear_scan_row_gates(q, k, v, heads=heads, dim=d, vdim=d, decay=decay, gain=gain, state=state, norm_state=norm_state,
+                                            q_start=q_start, slots=slots, q_scale=d ** -0.5),
+            lambda: S.linear_scan(q, k, v, **sizes, decay=const), moved + 8.0 * entries * heads * d, moved)
+        out[f"scan_channel_decay_{n}_tokens_{entries}_requests"] = beside(
+            lambda: S.linear_scan(q, k, v, **sizes, gate=gate, q_scale=d ** -0.5),
+            lambda: S.linear_scan(q, k, v, **sizes, gate=gate, beta=beta), moved + n * vw * 4, moved + n * vw * 4)
+    # what the scans read, and the read-outs, beside the delta rule's preparation and gated norm
+    for n, entries in ((2048, 1), (32, 32)):
+        q_start, slots = ints(list(range(0, n + 1, n // entries))), ints(list(range(entries)))
+        entry = ints([e for e in range(entries) for _ in range(n // entries)])
+        proj = bf(n, 4 * vw + 2 * heads)
+        m_state, bias = torch.zeros(entries + 1, heads, device=dev), f32(heads)
+        decay_rank = 16
+        delta_proj, up, up_bias = bf(n, 3 * vw + heads + 2 * d // 4), bf(decay_rank, vw), f32(vw)
+        taps, conv = f32(3 * vw, 4), torch.zeros(entries + 1, 3, 3 * vw, device=dev)
+        delta_up = bf(d // 4, vw)
+        prepare = lambda: S.delta_prepare(delta_proj, heads=heads, qk_heads=heads, dim=d, vdim=d, beta_offset=3 * vw, low_offset=3 * vw + heads,
+                                          rank=d // 4, taps=taps, conv_state=conv, a_log=bias, dt_bias=up_bias, a_up=delta_up, q_start=q_start,
+                                          slots=slots, token_entry=entry, unit_eps=1e-6, q_scale=1.0)
+        out[f"memory_gates_{n}_tokens"] = beside(
+            lambda: S.memory_gates(proj, heads=heads, i_offset=4 * vw, f_offset=4 * vw + heads, i_bias=bias, f_bias=bias, cap=15.0, m_state=m_state,
+                                   q_start=q_start, slots=slots), prepare, n * heads * 16, n * vw * 22)
+        out[f"channel_decay_{n}_tokens"] = beside(
+            lambda: S.channel_decay(proj, up, up_bias, offset=4 * vw, tau=16.0), prepare, n * vw * 4, n * vw * 22)
+        x, w, w_all = f32(n, vw), f32(d), f32(vw)
+        den, floor = f32(n, heads), torch.rand(n, heads, device=dev) + 0.1
+        gate_offset = 3 * vw
+        like = lambda: S.group_norm_gate(x, w, 1e-6, proj, gate_offset=gate_offset, out_dtype=torch.bfloat16)
+        out[f"read_out_memory_{n}_tokens"] = beside(
+            lambda: S.group_norm_gate(x, w_all, 1e-6, proj, gate_offset=gate_offset, group=d, divisor=(den, floor, 1e-6), out_dtype=torch.bfloat16),
+            like, n * vw * 8)
+        out[f"read_out_linear_{n}_tokens"] = beside(
+            lambda: S.group_norm_gate(x, w, 1e-6, proj, gate_offset=gate_offset, act="silu", out_dtype=torch.bfloat16), like, n * vw * 8)
+    # the gated unit in the projections' epilogues: gelu beside SiLU
+    gate_up = bf(2 * ff, width)
+    for n in (2048, 8):
+        x = bf(n, width)
+        linear = gemm_bf16.linear if n >= 128 else gemm_bf16.linear_skinny
+        out[f"gated_projection_{n}_tokens"] = beside(
+            lambda: linear(x, gate_up, None, torch.bfloat16, swiglu="gelu_tanh"), lambda: linear(x, gate_up, None, torch.bfloat16, swiglu=True),
+            None if n > 8 else 2 * ff * width * 2, flops=4.0 * n * ff * width)
+    # the embedding with its norm beside the same sum without one; rotations in either pairing; gates per head; soft cap
+    vocab, buckets = 32000, 65521
+    tables, norm_w = (bf(vocab, width), bf(buckets + 1, width)), f32(width)
+    for n, entries in ((2048, 1), (32, 32)):
+        ids = torch.randint(0, vocab, (n,), dtype=torch.int32, device=dev)
+        per = n // entries
+        positions, entry = ints([j + 1 for _ in range(entries) for j in range(per)]), ints([e for e in range(entries) for _ in range(per)])
+        q_start, slots = ints(list(range(0, n + 1, per))), ints(list(range(entries)))
+        previous = torch.zeros(entries + 1, 1, dtype=torch.int32, device=dev)
+        embed = lambda **more: F.embedding_sum(ids, *tables, positions=positions, token_entry=entry, q_start=q_start, slots=slots, previous=previous,
+                                               freq=None, buckets=buckets, mul_prev=131, mul_cur=17, scale=64.0, **more)
+        out[f"embedding_{n}_tokens"] = beside(lambda: embed(norm=(norm_w, 1e-6), rounded_dtype=torch.bfloat16), embed, n * width * 10, n * width * 8)
+        q_rank, inv_freq = width // 2, torch.rand(rot // 2, device=dev)
+        rows, qw, kw = bf(n, q_rank + rank + rot + heads), f32(q_rank), f32(rank)
+        table = torch.arange(n // page + entries, dtype=torch.int32).repeat(entries, 1).to(dev)
+        pool = bf(n // page + entries, page, rank + rot)
+        latent = lambda **more: M.latent_prepare(rows, q_offset=0, q_rank=q_rank, q_weight=qw, eps=1e-6, positions=positions, token_entry=entry,
+                                                 kv_offset=q_rank, kv_rank=rank, kv_weight=kw, rot=rot, rot_dims=rot, inv_freq=inv_freq,
+                                                 block_table=table, page_size=page, pool=pool, **more)
+        out[f"latent_rows_{n}_tokens"] = beside(lambda: latent(interleaved=True, rot_factor=1.2), latent, n * (q_rank + rank + rot) * 4)
+        q, absorbed = bf(n, heads * (d + rot)), bf(n, heads * (rank + rot))
+        turn = lambda **more: M.rope_slice(q, absorbed, heads=heads, src_head=d + rot, src_offset=d, dst_head=rank + rot, dst_offset=rank, rot=rot,
+                                           rot_dims=rot, inv_freq=inv_freq, positions=positions, **more)
+        out[f"rotation_{n}_tokens"] = beside(lambda: turn(interleaved=True, rot_factor=1.2), turn, n * heads * rot * 4)
+        attn, gates = bf(n, vw), bf(n, vw)
+        out[f"gate_per_head_{n}_tokens"] = beside(lambda: M.sigmoid_gate(attn, gates, gate_offset=0, group=d),
+                                                  lambda: M.sigmoid_gate(attn, gates, gate_offset=0, group=1), n * vw * 4, n * vw * 6)
+        x, resid = f32(n, width), f32(n, width)
+        out[f"norm_on_output_{n}_tokens"] = beside(lambda: M.norm_accumulate_round(x, norm_w, 1e-6, resid, torch.bfloat16, 0.5),
+                                                   lambda: F.add_rmsnorm(resid, x, norm_w, 1e-6, torch.bfloat16), n * width * 14)
+    logits, like = f32(32, 151936), bf(32, 2 * 151936)
+    out["soft_cap_32_tokens"] = beside(lambda: F.soft_cap(logits, 30.0), lambda: F.relu2(like), logits.numel() * 8)
+    return out
+
+
 def run_reference(args) -> dict:
     """The unmodified reference from baseline/_ref: its own Qwen3ForCausalLM, paged cache,
     CUDA-graph decode and BatchScheduler, driven through Engine.create_scheduler()."""
@@ -1415,13 +1601,14 @@ def main() -> int:
     parser.add_argument("--batch", type=int, default=8)
     parser.add_argument("--context", type=int, default=0, help="with --only decode: cached tokens per request (default 2048)")
     parser.add_argument("--layers", type=int, default=0, help="fewer layers than the configuration has (named in config)")
-    parser.add_argument("--workload", choices=("default", "staggered14b", "decode32b", "sorulix", "ropulix", "mabedra", "tafisun"), default="default",
+    parser.add_argument("--workload", choices=("default", "staggered14b", "decode32b", "sorulix", "ropulix", "mabedra", "tafisun", "fumolorn"), default="default",
                         help="default: Qwen3-8B decode/prefill; staggered14b, decode32b: the larger configurations (either --impl); "
                              "sorulix: the Sorulix design beside Qwen3 at equal sizes, and its kernels alone; "
                              "ropulix: the Ropulix design beside Sorulix and Qwen3 at equal sizes, and its kernels alone; "
                              "mabedra: the Mabedra design beside Qwen3 and Ropulix at equal sizes, and its kernels alone; "
-                             "tafisun: the Tafisun design beside Ropulix and Qwen3 at equal sizes, and its kernels alone")
-    parser.add_argument("--size", default="", help="with --workload sorulix, ropulix, mabedra or tafisun: sizes to run, with commas (2k, 4k; default both)")
+                             "tafisun: the Tafisun design beside Ropulix and Qwen3 at equal sizes, and its kernels alone; "
+                             "fumolorn: the Fumolorn design beside Ropulix, Sorulix and Qwen3 at equal sizes, and its kernels alone")
+    parser.add_argument("--size", default="", help="with --workload sorulix, ropulix, mabedra, tafisun or fumolorn: sizes to run, with commas (2k, 4k; default both)")
     parser.add_argument("--only", choices=("all", "decode", "prefill", "kernels", "models"), default="all",
                         help="run only the decode steps or only the prefill (for profiler captures of a small case); "
                              "with --workload sorulix: only the kernels alone, or only the whole models")
@@ -1453,6 +1640,11 @@ def main() -> int:
             result = _unavailable("the reference has no model of this design")
         else:
             result = run_tafisun(args)
+    elif args.workload == "fumolorn":
+        if args.impl == "reference":
+            result = _unavailable("the reference has no model of this design")
+        else:
+            result = run_fumolorn(args)
     else:
         result = run_reference(args) if args.impl == "reference" else run_ours(args)
     print(json.dumps(result))

@@ -411,33 +411,48 @@ memory_gates_kernel(const T* __restrict__ proj, int ld, int i_off, int f_off, co
   float* kept = m_state + static_cast<size_t>(slots[entry]) * H + h;
   const float bi = i_bias[h], bf = f_bias[h];
   float m = *kept;
-  float zi = 0.f, zf = 0.f;
-  auto fetch = [&](int t) {
+  // the logits of the chunk of 32 tokens in hand and of the kAhead - 1 behind it: a fetch takes longer than a chunk's chain
+  constexpr int kAhead = 4;
+  float zi[kAhead], zf[kAhead];
+  auto fetch = [&](int t, int at) {
+    zi[at] = zf[at] = 0.f;
     if (t < t_end) {
-      zi = to_float(proj[static_cast<size_t>(t) * ld + i_off + h]);
-      zf = to_float(proj[static_cast<size_t>(t) * ld + f_off + h]);
+      zi[at] = to_float(proj[static_cast<size_t>(t) * ld + i_off + h]);
+      zf[at] = to_float(proj[static_cast<size_t>(t) * ld + f_off + h]);
     }
   };
-  fetch(t_begin + lane);
-  for (int t0 = t_begin; t0 < t_end; t0 += 32) {
-    const float li = cap * tanhf((zi + bi) / cap), lf = log_sigmoid_f(cap * tanhf((zf + bf) / cap));
-    fetch(t0 + 32 + lane);
-    const int count = min(32, t_end - t0);
-    float before = 0.f, after = 0.f;
-    for (int j = 0; j < count; ++j) {
-      const float fj = __shfl_sync(0xffffffffu, lf, j), ij = __shfl_sync(0xffffffffu, li, j);
-      const float m_new = fmaxf(fj + m, ij);
-      if (lane == j) {
-        before = m;
-        after = m_new;
+#pragma unroll
+  for (int c = 0; c < kAhead; ++c) fetch(t_begin + 32 * c + lane, c);
+  for (int base = t_begin; base < t_end; base += 32 * kAhead) {
+#pragma unroll
+    for (int c = 0; c < kAhead; ++c) {
+      const int t0 = base + 32 * c;
+      if (t0 >= t_end) break;
+      const float li = cap * tanhf((zi[c] + bi) / cap), lf = log_sigmoid_f(cap * tanhf((zf[c] + bf) / cap));
+      fetch(t0 + 32 * kAhead + lane, c);
+      const int count = min(32, t_end - t0);
+      float before = 0.f, after = 0.f;
+      auto step = [&](int j) {
+        const float fj = __shfl_sync(0xffffffffu, lf, j), ij = __shfl_sync(0xffffffffu, li, j);
+        const float m_new = fmaxf(fj + m, ij);
+        if (lane == j) {
+          before = m;
+          after = m_new;
+        }
+        m = m_new;
+      };
+      if (count == 32) {       // unrolled: the shuffles of later tokens do not wait for the chain
+#pragma unroll
+        for (int j = 0; j < 32; ++j) step(j);
+      } else {
+        for (int j = 0; j < count; ++j) step(j);
       }
-      m = m_new;
-    }
-    if (lane < count) {
-      const size_t at = static_cast<size_t>(t0 + lane) * H + h;
-      decay[at] = expf(lf + before - after);
-      gain[at] = expf(li - after);
-      floor_[at] = expf(-after);
+      if (lane < count) {
+        const size_t at = static_cast<size_t>(t0 + lane) * H + h;
+        decay[at] = expf(lf + before - after);
+        gain[at] = expf(li - after);
+        floor_[at] = expf(-after);
+      }
     }
   }
   if (lane == 0) *kept = m;
