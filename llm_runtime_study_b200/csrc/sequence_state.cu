@@ -409,17 +409,18 @@ memory_gates_kernel(const T* __restrict__ proj, int ld, int i_off, int f_off, co
   if (h >= H) return;
   const int t_end = q_start[entry + 1], t_begin = q_start[entry];
   float* kept = m_state + static_cast<size_t>(slots[entry]) * H + h;
+  if (t_end <= t_begin) return;
   const float bi = i_bias[h], bf = f_bias[h];
   float m = *kept;
   // the logits of the chunk of 32 tokens in hand and of the kAhead - 1 behind it: a fetch takes longer than a chunk's chain
   constexpr int kAhead = 4;
-  float zi[kAhead], zf[kAhead];
+  // (kept in the storage type and fetched without a branch, so that nothing waits for a load before its chunk comes up; a
+  // lane past the end reads the last token again, and nothing is made of that)
+  T zi[kAhead], zf[kAhead];
   auto fetch = [&](int t, int at) {
-    zi[at] = zf[at] = 0.f;
-    if (t < t_end) {
-      zi[at] = to_float(proj[static_cast<size_t>(t) * ld + i_off + h]);
-      zf[at] = to_float(proj[static_cast<size_t>(t) * ld + f_off + h]);
-    }
+    const T* row = proj + static_cast<size_t>(min(t, t_end - 1)) * ld + h;
+    zi[at] = row[i_off];
+    zf[at] = row[f_off];
   };
 #pragma unroll
   for (int c = 0; c < kAhead; ++c) fetch(t_begin + 32 * c + lane, c);
@@ -428,7 +429,8 @@ memory_gates_kernel(const T* __restrict__ proj, int ld, int i_off, int f_off, co
     for (int c = 0; c < kAhead; ++c) {
       const int t0 = base + 32 * c;
       if (t0 >= t_end) break;
-      const float li = cap * tanhf((zi[c] + bi) / cap), lf = log_sigmoid_f(cap * tanhf((zf[c] + bf) / cap));
+      const float li = cap * tanhf((to_float(zi[c]) + bi) / cap);
+      const float lf = log_sigmoid_f(cap * tanhf((to_float(zf[c]) + bf) / cap));
       fetch(t0 + 32 * kAhead + lane, c);
       const int count = min(32, t_end - t0);
       float before = 0.f, after = 0.f;
