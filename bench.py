@@ -1318,18 +1318,18 @@ def _fumolorn_config(width, ff, heads, kv_heads, d, pairs, vocab) -> dict:
     recurrences keep ``heads`` states of ``d x d`` and the latent rows are as wide as in the Ropulix configuration."""
 
     latent = {"heads": heads, "dim": d, "rot_dim": d // 2, "vdim": d, "kv_rank": 4 * d, "q_rank": width // 2, "scale": (d + d // 2) ** -0.5,
-              "rot": {"base": 50000.0, "dims": d // 2, "scaling": {"factor": 8.0, "original": 1024, "fast": 32.0, "slow": 1.0}}}
+              "rot": {"base": 10000.0, "dims": d // 2, "scaling": {"factor": 4.0, "original": 4096, "fast": 24.0, "slow": 2.0}}}
     mlp = {"kind": "dense", "ff": ff}
     layers = []
     for _ in range(pairs):
         layers += [
-            {"type": "gla", "mixer": {"heads": heads, "dim": d, "vdim": d, "tau": 16.0}, "mlp": mlp},
+            {"type": "gla", "mixer": {"heads": heads, "dim": d, "vdim": d, "tau": 8.0}, "mlp": mlp},
             {"type": "latent_attention", "mixer": latent, "mlp": mlp},
             {"type": "mlstm", "mixer": {"heads": heads, "dim": d, "vdim": d, "gate_cap": 15.0}, "mlp": mlp},
             {"type": "latent_attention", "mixer": latent, "mlp": mlp},
         ]
     return {"architecture": "Fumolorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "torch_dtype": "bfloat16",
-            "residual_mult": 0.5, "logit_softcap": 30.0, "layers": layers[: 2 * pairs],
+            "residual_mult": 0.5, "logit_softcap": 25.0, "layers": layers[: 2 * pairs],
             "embedding": {"scale": width ** 0.5, "bigram": {"buckets": 65521, "mul_prev": 131, "mul_cur": 17}}}
 
 

@@ -21,8 +21,7 @@ from ..errors import ConfigError
 from .description import LayerDescription, ModelDescription
 from .tafisun import stored_name
 
-MLP_ACT = "gelu_tanh"        # fixed by the design (not in config.json)
-DEFAULT_DECAY_RANK = 16      # what random weights are drawn with: only a stored tensor's shape gives a gla layer's decay rank
+MLP_ACT = "gelu_tanh"     # fixed by the design (not in config.json)
 
 
 def _mixer(index: int, layer: FumolornLayer, config: FumolornConfig, ranks: dict[int, int]) -> dict:
@@ -31,7 +30,7 @@ def _mixer(index: int, layer: FumolornLayer, config: FumolornConfig, ranks: dict
     if isinstance(m, MatrixMemory):
         return {"kind": "matrix_memory", **sizes, "gate_cap": m.gate_cap}
     if isinstance(m, GatedLinear):
-        return {"kind": "gated_linear_attention", **sizes, "tau": m.tau, "decay_rank": ranks.get(index, DEFAULT_DECAY_RANK)}
+        return {"kind": "gated_linear_attention", **sizes, "tau": m.tau, "decay_rank": ranks.get(index, max(1, m.dim // 4))}
     assert isinstance(m, LatentAttention)
     q_rank = m.q_rank or ranks.get(index, 0)
     if q_rank <= 0:
@@ -46,7 +45,8 @@ def _mixer(index: int, layer: FumolornLayer, config: FumolornConfig, ranks: dict
 
 def describe_fumolorn(config: FumolornConfig, ranks: dict[int, int] | None = None) -> ModelDescription:
     """``ranks``: per layer, the inner size of a low-rank map that config.json does not give (a gla layer's decay; a latent
-    attention layer's query where the configuration leaves it out): the stored tensors' shapes do (``describe_for_checkpoint``)."""
+    attention layer's query where the configuration leaves it out): the stored tensors' shapes do (``describe_for_checkpoint``).
+    Without them a quarter of the key size is assumed for the decay, which is what random weights are drawn with."""
 
     norm = {"kind": "rms_norm", "dim": config.width, "eps": config.eps}
     layers = []
