@@ -2,6 +2,7 @@ from .fields import read_config_dict, required, optional
 from .fumolorn import FumolornConfig
 from .mabedra import MabedraConfig
 from .qwen3 import Qwen3Config
+from .refolix import RefolixConfig
 from .ropulix import RopulixConfig
 from .sorulix import SorulixConfig
 from .tafisun import TafisunConfig
@@ -18,6 +19,7 @@ __all__ = [
     "FumolornConfig",
     "MabedraConfig",
     "Qwen3Config",
+    "RefolixConfig",
     "RopulixConfig",
     "SorulixConfig",
     "TafisunConfig",

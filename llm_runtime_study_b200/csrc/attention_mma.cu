@@ -1,5 +1,5 @@
 // bfloat16 tensor-core attention over the paged cache, built once per head size
-// (-DHEAD_DIM=<multiple of 16, at most 256>).
+// (-DHEAD_DIM=<multiple of 16, at most 256>; -DVALUE_DIM=<the same> where the values' head size is another one than the keys').
 //
 //   prefill kernel  a tile of up to TM consecutive query tokens of one request times the
 //                   query heads that share one KV head forms the rows of S = Q K^T; keys
@@ -27,17 +27,23 @@
 #ifndef HEAD_DIM
 #error "compile with -DHEAD_DIM=<head size>"
 #endif
+#ifndef VALUE_DIM
+#define VALUE_DIM HEAD_DIM
+#endif
+static_assert(VALUE_DIM % 16 == 0 && VALUE_DIM >= 16 && VALUE_DIM <= 256, "the values' head size must be 16..256 in steps of 16");
 static_assert(HEAD_DIM % 16 == 0 && HEAD_DIM >= 16 && HEAD_DIM <= 256, "head size must be 16..256 in steps of 16");
 
 namespace b200 {
 
 using bf16 = __nv_bfloat16;
-constexpr int D = HEAD_DIM;
+constexpr int D = HEAD_DIM;       // columns of q and k
+constexpr int DV = VALUE_DIM;     // columns of v and of the output
 constexpr int BN = 64;            // keys per shared-memory tile
 constexpr int LDS = D + 8;        // padded row length: ldmatrix rows fall into different banks
+constexpr int LDV = DV + 8;
 constexpr int KSTEPS = D / 16;    // 16-wide steps over the head size in Q K^T
-constexpr int DTILES = D / 8;     // 8-wide column tiles of the output
-constexpr int kSmemBytes = 2 * 2 * BN * LDS * 2;
+constexpr int DTILES = DV / 8;    // 8-wide column tiles of the output
+constexpr int kSmemBytes = 2 * BN * (LDS + LDV) * 2;
 
 struct AttnParams {
   const bf16* q;
@@ -65,7 +71,7 @@ struct AttnParams {
   // decode
   const int* kv_len;
   int num_splits;
-  float* part_o;   // [B][nq][splits][D]
+  float* part_o;   // [B][nq][splits][DV]
   float* part_ml;  // [B][nq][splits][2]
 };
 
@@ -74,26 +80,32 @@ struct AttnParams {
 template <int NT>
 __device__ __forceinline__ void load_kv_tile(bf16* ks, bf16* vs, const AttnParams& p, const int* table,
                                              int kvh, int t0, int lo, int hi) {
-  constexpr int CH = D / 8;
-  for (int c = threadIdx.x; c < BN * CH; c += NT) {
-    const int r = c / CH, ch = c - r * CH;
+  // a row's chunks of 16 bytes: the first CH of them hold its key (and, of equal size, its value beside it), those behind
+  // them, where the sizes differ, its value
+  constexpr int CH = D / 8, CV = D == DV ? 0 : DV / 8;
+  for (int c = threadIdx.x; c < BN * (CH + CV); c += NT) {
+    const int r = c / (CH + CV), ch = c - r * (CH + CV);
     const int t = t0 + r;
-    const bf16* ksrc = p.k_pool;
-    const bf16* vsrc = p.v_pool;
+    size_t row = 0;
     int bytes = 0;
     if (t >= lo && t <= hi) {
       const int index = p.page_shift >= 0 ? t >> p.page_shift : t / p.page_size;
       const int slot = p.page_shift >= 0 ? t & (p.page_size - 1) : t - index * p.page_size;
       const int page = table[index];
       if (page >= 0) {
-        const size_t off = ((static_cast<size_t>(page) * p.nkv + kvh) * p.page_size + slot) * D + ch * 8;
-        ksrc += off;
-        vsrc += off;
+        row = (static_cast<size_t>(page) * p.nkv + kvh) * p.page_size + slot;
         bytes = 16;
       }
     }
-    cp_async_16(ks + r * LDS + ch * 8, ksrc, bytes);
-    cp_async_16(vs + r * LDS + ch * 8, vsrc, bytes);
+    if constexpr (CV == 0) {
+      const size_t off = bytes ? row * D + ch * 8 : 0;
+      cp_async_16(ks + r * LDS + ch * 8, p.k_pool + off, bytes);
+      cp_async_16(vs + r * LDV + ch * 8, p.v_pool + off, bytes);
+    } else if (ch < CH) {
+      cp_async_16(ks + r * LDS + ch * 8, p.k_pool + (bytes ? row * D + ch * 8 : 0), bytes);
+    } else {
+      cp_async_16(vs + r * LDV + (ch - CH) * 8, p.v_pool + (bytes ? row * DV + (ch - CH) * 8 : 0), bytes);
+    }
   }
 }
 
@@ -197,7 +209,7 @@ __device__ __forceinline__ void warp_attend(const bf16* kbuf, const bf16* vbuf, 
 #pragma unroll
     for (int dtp = 0; dtp < DTILES / 2; ++dtp) {
       uint32_t vf[4];
-      ldmatrix_x4_trans(vf, vbuf + (key0 + kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LDS + dtp * 16 + ((lane >> 4) & 1) * 8);
+      ldmatrix_x4_trans(vf, vbuf + (key0 + kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LDV + dtp * 16 + ((lane >> 4) & 1) * 8);
       mma_bf16(o[2 * dtp], a, vf[0], vf[1]);
       mma_bf16(o[2 * dtp + 1], a, vf[2], vf[3]);
     }
@@ -234,7 +246,7 @@ __global__ void __launch_bounds__(WARPS * 32) prefill_attention_kernel(AttnParam
 
   bool row_ok[2];
   int row_hi[2], row_lo[2];
-  long row_off[2];
+  long row_off[2], out_off[2];
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     const int R = warp * 16 + gid + i * 8;
@@ -244,6 +256,7 @@ __global__ void __launch_bounds__(WARPS * 32) prefill_attention_kernel(AttnParam
     row_lo[i] = p.window > 0 ? max(0, row_hi[i] - p.window + 1) : 0;
     if (RULES && p.chunk > 0) row_lo[i] = max(row_lo[i], row_hi[i] / p.chunk * p.chunk);
     row_off[i] = (static_cast<long>(tok0 + tl) * p.nq + kvh * p.group + g) * D;
+    out_off[i] = (static_cast<long>(tok0 + tl) * p.nq + kvh * p.group + g) * DV;
   }
   ScoreRules rules{};
   if constexpr (RULES) {
@@ -280,7 +293,7 @@ __global__ void __launch_bounds__(WARPS * 32) prefill_attention_kernel(AttnParam
   for (int j = 0; j < ntiles; ++j) {
     const int buf = j & 1;
     if (j + 1 < ntiles) {
-      load_kv_tile<WARPS * 32>(ks + (buf ^ 1) * BN * LDS, vs + (buf ^ 1) * BN * LDS, p, table, kvh,
+      load_kv_tile<WARPS * 32>(ks + (buf ^ 1) * BN * LDS, vs + (buf ^ 1) * BN * LDV, p, table, kvh,
                                t_begin + (j + 1) * BN, lo, p_last);
       cp_async_commit();
       cp_async_wait<1>();
@@ -288,7 +301,7 @@ __global__ void __launch_bounds__(WARPS * 32) prefill_attention_kernel(AttnParam
       cp_async_wait<0>();
     }
     __syncthreads();
-    warp_attend<BN / 8, RULES>(ks + buf * BN * LDS, vs + buf * BN * LDS, 0, t_begin + j * BN, qf, row_ok, row_hi, row_lo,
+    warp_attend<BN / 8, RULES>(ks + buf * BN * LDS, vs + buf * BN * LDV, 0, t_begin + j * BN, qf, row_ok, row_hi, row_lo,
                                p.scale_log2, m, l, o, &rules);
     __syncthreads();
   }
@@ -298,7 +311,7 @@ __global__ void __launch_bounds__(WARPS * 32) prefill_attention_kernel(AttnParam
     float total = quad_sum(l[i]);
     if (RULES && p.sink) total += exp2f(-m[i]);     // the sink's exp(0 - maximum); no visible key: infinity, a row of zeros
     const float inv = total > 0.f ? 1.f / total : 0.f;
-    bf16* dst = p.out + row_off[i];
+    bf16* dst = p.out + out_off[i];
 #pragma unroll
     for (int dt = 0; dt < DTILES; ++dt)
       *reinterpret_cast<uint32_t*>(dst + dt * 8 + tig * 2) = pack_bf16(o[dt][2 * i] * inv, o[dt][2 * i + 1] * inv);
@@ -367,32 +380,36 @@ __global__ void __launch_bounds__(128) decode_attention_kernel(AttnParams p) {
   // the loop, so the warps drift apart and cover each other's waits.
   constexpr int WB = 16;                                  // keys per warp block
   bf16* wk = ks + warp * (2 * WB * LDS);                  // [2][WB][LDS] keys
-  bf16* wv = vs + warp * (2 * WB * LDS);                  // [2][WB][LDS] values
+  bf16* wv = vs + warp * (2 * WB * LDV);                  // [2][WB][LDV] values
   const int nblocks = c1 >= c0 ? (c1 - c0) / WB + 1 : 0;  // 16-key blocks in this CTA's part
   const int hi_here[2] = {min(row_hi[0], c1), min(row_hi[1], c1)};
   auto load_block = [&](int block, int buf) {
-    constexpr int CH = D / 8;
+    constexpr int CH = D / 8, CV = D == DV ? 0 : DV / 8;       // as in load_kv_tile
     const int t0 = c0 + block * WB;
 #pragma unroll
-    for (int c = lane; c < WB * CH; c += 32) {
-      const int r = c / CH, ch = c - r * CH;
+    for (int c = lane; c < WB * (CH + CV); c += 32) {
+      const int r = c / (CH + CV), ch = c - r * (CH + CV);
       const int t = t0 + r;
-      const bf16* ksrc = p.k_pool;
-      const bf16* vsrc = p.v_pool;
+      size_t row = 0;
       int bytes = 0;
       if (t <= c1) {
         const int index = p.page_shift >= 0 ? t >> p.page_shift : t / p.page_size;
         const int slot = p.page_shift >= 0 ? t & (p.page_size - 1) : t - index * p.page_size;
         const int page = table[index];
         if (page >= 0) {
-          const size_t off = ((static_cast<size_t>(page) * p.nkv + kvh) * p.page_size + slot) * D + ch * 8;
-          ksrc += off;
-          vsrc += off;
+          row = (static_cast<size_t>(page) * p.nkv + kvh) * p.page_size + slot;
           bytes = 16;
         }
       }
-      cp_async_16(wk + (buf * WB + r) * LDS + ch * 8, ksrc, bytes);
-      cp_async_16(wv + (buf * WB + r) * LDS + ch * 8, vsrc, bytes);
+      if constexpr (CV == 0) {
+        const size_t off = bytes ? row * D + ch * 8 : 0;
+        cp_async_16(wk + (buf * WB + r) * LDS + ch * 8, p.k_pool + off, bytes);
+        cp_async_16(wv + (buf * WB + r) * LDV + ch * 8, p.v_pool + off, bytes);
+      } else if (ch < CH) {
+        cp_async_16(wk + (buf * WB + r) * LDS + ch * 8, p.k_pool + (bytes ? row * D + ch * 8 : 0), bytes);
+      } else {
+        cp_async_16(wv + (buf * WB + r) * LDV + (ch - CH) * 8, p.v_pool + (bytes ? row * DV + (ch - CH) * 8 : 0), bytes);
+      }
     }
   };
   if (warp < nblocks) {
@@ -409,7 +426,7 @@ __global__ void __launch_bounds__(128) decode_attention_kernel(AttnParams p) {
       cp_async_wait<0>();
     }
     __syncwarp();
-    warp_attend<2, RULES>(wk + buf * WB * LDS, wv + buf * WB * LDS, 0, c0 + block * WB, qf, row_ok, hi_here, row_lo,
+    warp_attend<2, RULES>(wk + buf * WB * LDS, wv + buf * WB * LDV, 0, c0 + block * WB, qf, row_ok, hi_here, row_lo,
                           p.scale_log2, m, l, o, &rules);
     __syncwarp();
   }
@@ -418,7 +435,7 @@ __global__ void __launch_bounds__(128) decode_attention_kernel(AttnParams p) {
   // combine the four warps through shared memory (the K/V buffers are free now)
   float* sm_m = reinterpret_cast<float*>(smem_raw);  // [4][16]
   float* sm_l = sm_m + 64;                           // [4][16]
-  float* sm_o = sm_l + 64;                           // [4][16][D]
+  float* sm_o = sm_l + 64;                           // [4][16][DV]
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     const int R = gid + i * 8;
@@ -429,13 +446,13 @@ __global__ void __launch_bounds__(128) decode_attention_kernel(AttnParams p) {
     }
 #pragma unroll
     for (int dt = 0; dt < DTILES; ++dt) {
-      sm_o[(warp * 16 + R) * D + dt * 8 + tig * 2] = o[dt][2 * i];
-      sm_o[(warp * 16 + R) * D + dt * 8 + tig * 2 + 1] = o[dt][2 * i + 1];
+      sm_o[(warp * 16 + R) * DV + dt * 8 + tig * 2] = o[dt][2 * i];
+      sm_o[(warp * 16 + R) * DV + dt * 8 + tig * 2 + 1] = o[dt][2 * i + 1];
     }
   }
   __syncthreads();
-  for (int idx = threadIdx.x; idx < p.gs * D; idx += 128) {
-    const int R = idx / D, col = idx - R * D;
+  for (int idx = threadIdx.x; idx < p.gs * DV; idx += 128) {
+    const int R = idx / DV, col = idx - R * DV;
     const int g = slice * p.gs + R;
     if (g >= p.group) continue;
     float M = -INFINITY;
@@ -446,16 +463,16 @@ __global__ void __launch_bounds__(128) decode_attention_kernel(AttnParams p) {
 #pragma unroll
     for (int w = 0; w < 4; ++w) {
       const float f = exp2f(sm_m[w * 16 + R] - base);
-      acc += sm_o[(w * 16 + R) * D + col] * f;
+      acc += sm_o[(w * 16 + R) * DV + col] * f;
       L += sm_l[w * 16 + R] * f;
     }
     const int head = kvh * p.group + g;
     if (p.num_splits == 1) {
       if (RULES && p.sink) L += exp2f(-base);
-      p.out[(static_cast<long>(b) * p.nq + head) * D + col] = __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
+      p.out[(static_cast<long>(b) * p.nq + head) * DV + col] = __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
     } else {
       const long slot = (static_cast<long>(b) * p.nq + head) * p.num_splits + split;
-      p.part_o[slot * D + col] = acc;
+      p.part_o[slot * DV + col] = acc;
       if (col == 0) {
         p.part_ml[slot * 2] = M;
         p.part_ml[slot * 2 + 1] = L;
@@ -478,7 +495,7 @@ __global__ void __launch_bounds__(128) decode_attention_kernel(AttnParams p) {
 // two-stage buffer per warp) and is read transposed by ldmatrix.trans; P^T reaches the
 // B-fragment layout with movmatrix.trans.
 // grid (splits, nkv * slices, requests); at most 8 query heads of a group per CTA.
-#if HEAD_DIM % 32 == 0
+#if HEAD_DIM % 32 == 0 && VALUE_DIM == HEAD_DIM
 constexpr int kTGs = 8;                       // query heads per CTA = the N side of one mma
 constexpr int TLDS = D + 8;                   // padded V row
 constexpr int kTSmemBytes = 4 * 2 * 16 * TLDS * 2 > (2 * 4 * 8 + 4 * 8 * D) * 4 ? 4 * 2 * 16 * TLDS * 2 : (2 * 4 * 8 + 4 * 8 * D) * 4;
@@ -673,9 +690,9 @@ __global__ void __launch_bounds__(128) decode_attention_t_kernel(AttnParams p) {
   }
 }
 
-#endif  // HEAD_DIM % 32 == 0
+#endif  // HEAD_DIM % 32 == 0 && VALUE_DIM == HEAD_DIM
 
-// grid (nq, requests), D threads: combine the splits of one (request, head)
+// grid (nq, requests), DV threads: combine the splits of one (request, head)
 __global__ void decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                     bf16* __restrict__ out, int nq, int num_splits, int sink) {
   pdl_trigger();
@@ -684,19 +701,19 @@ __global__ void decode_merge_kernel(const float* __restrict__ part_o, const floa
   float M = -INFINITY;
   for (int s = 0; s < num_splits; ++s) M = fmaxf(M, part_ml[(base + s) * 2]);
   const float ref = M == -INFINITY ? 0.f : M;
-  for (int col = threadIdx.x; col < D; col += blockDim.x) {
+  for (int col = threadIdx.x; col < DV; col += blockDim.x) {
     float acc = 0.f, L = 0.f;
     for (int s = 0; s < num_splits; ++s) {
       const float f = exp2f(part_ml[(base + s) * 2] - ref);
-      acc += part_o[(base + s) * D + col] * f;
+      acc += part_o[(base + s) * DV + col] * f;
       L += part_ml[(base + s) * 2 + 1] * f;
     }
     if (sink) L += exp2f(-ref);      // the sink's exp(0 - maximum), once for all parts
-    out[(static_cast<long>(blockIdx.y) * nq + blockIdx.x) * D + col] = __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
+    out[(static_cast<long>(blockIdx.y) * nq + blockIdx.x) * DV + col] = __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
   }
 }
 
-constexpr int kMergeThreads = D < 128 ? D : 128;
+constexpr int kMergeThreads = DV < 128 ? DV : 128;
 static int heads_per_cta(int group) { return group < 16 ? group : 16; }
 
 }  // namespace b200
@@ -729,6 +746,7 @@ static int fill_common(AttnParams& p, const void* q, const void* k_pool, const v
 }
 
 extern "C" int b200_attention_head_dim() { return HEAD_DIM; }
+extern "C" int b200_attention_value_dim() { return VALUE_DIM; }
 
 // Rows per CTA of the prefill kernel: the caller cuts entries into tiles of
 // tokens_per_tile = rows / heads_per_cta consecutive tokens.
@@ -800,7 +818,7 @@ extern "C" int b200_attention_prefill_masked_bf16(const void* q, const void* k_p
 }
 
 extern "C" long b200_attention_decode_scratch_floats(int requests, int nq, int num_splits) {
-  return num_splits <= 1 ? 0 : static_cast<long>(requests) * nq * num_splits * (D + 2);
+  return num_splits <= 1 ? 0 : static_cast<long>(requests) * nq * num_splits * (DV + 2);
 }
 
 extern "C" int b200_attention_decode_bf16(const void* q, const void* k_pool, const void* v_pool, void* out,
@@ -815,8 +833,8 @@ extern "C" int b200_attention_decode_bf16(const void* q, const void* k_pool, con
   p.kv_len = kv_len;
   p.num_splits = num_splits;
   p.part_o = scratch;
-  p.part_ml = scratch + static_cast<long>(requests) * nq * num_splits * D;
-#if HEAD_DIM % 32 == 0
+  p.part_ml = scratch + static_cast<long>(requests) * nq * num_splits * DV;
+#if HEAD_DIM % 32 == 0 && VALUE_DIM == HEAD_DIM
   // The transposed kernel, unless LLM_RUNTIME_STUDY_B200_DECODE_ATTENTION=rows asks for the
   // older one with the query heads on the 16-row side (kept for head sizes like 48 and 80).
   static int use_rows = -1;
@@ -864,7 +882,7 @@ extern "C" int b200_attention_decode_masked_bf16(const void* q, const void* k_po
   p.kv_len = kv_len;
   p.num_splits = num_splits;
   p.part_o = scratch;
-  p.part_ml = scratch + static_cast<long>(requests) * nq * num_splits * D;
+  p.part_ml = scratch + static_cast<long>(requests) * nq * num_splits * DV;
   p.scale = scale;
   p.softcap = softcap;
   p.slopes = slopes;

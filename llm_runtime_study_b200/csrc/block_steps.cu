@@ -2,7 +2,7 @@
 // layer norm (mean and variance, a weight, no bias), a short causal convolution over time added to
 // what each sublayer reads (inputs before the step come from rows kept per request), the sum of the
 // scaled sublayer outputs into the stream together with a weighted average over the results of all
-// layers so far, a polynomial activation of normalised powers, and the gated unit of routed rows
+// layers so far, the norm of a scaled stream plus a sublayer's output, a polynomial activation of normalised powers, and the gated unit of routed rows
 // whose router weight multiplies the expert's input.  Statistics and sums are float32; the order of
 // every sum depends on the row's width or on the token's own position only.
 #include "common.cuh"
@@ -243,6 +243,130 @@ scale_sum_average_vec_kernel(float* __restrict__ x, const float* __restrict__ a,
   *reinterpret_cast<float4*>(x + i) = v;
 }
 
+// ------------------------------------------------------------- norm behind the sum
+// x = norm(alpha * x + s * y) * w in place on the float32 stream, one CTA per row; the norm subtracts the row's mean first
+// (`centred`: layer norm) or not (RMS norm), statistics in two passes over the row kept in shared memory.  `rounded` (optional)
+// receives the new row in the activation type, for the sublayer that reads it next.  s: one factor per column, or null.
+// y, the sublayer's output, is given in one of three forms:
+//   y != null, branches 0, pair_row null   rows of y
+//   pair_row != null                       sum_j pair_w[t, j] * y[pair_row[t, j]], j ascending (what a router's experts returned),
+//                                          plus extra_scale[t] * extra[t] where given (what runs for every token)
+//   branches 1 or 2                        factor * sum_b branch_b[t] * rsqrt(mean(branch_b[t]^2) + branch_eps) * branch_w_b
+struct SumNormArgs {
+  float* x;
+  const float* y;
+  const int* pair_row; const float* pair_w; int top;
+  const float* extra; const float* extra_scale;
+  const float* branch[2]; const float* branch_w[2]; int branches; float branch_eps, branch_factor;
+  const float* s; const float* w;
+  float alpha, eps;
+  int centred, hidden;
+};
+
+// V: float4 (hidden a multiple of 4, every row on a 16-byte boundary) or float.
+template <typename V> struct Lanes;
+template <> struct Lanes<float> {
+  static constexpr int n = 1;
+  __device__ static void get(const float& v, float* f) { f[0] = v; }
+  __device__ static float put(const float* f) { return f[0]; }
+};
+template <> struct Lanes<float4> {
+  static constexpr int n = 4;
+  __device__ static void get(const float4& v, float* f) { f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w; }
+  __device__ static float4 put(const float* f) { return make_float4(f[0], f[1], f[2], f[3]); }
+};
+template <typename V> __device__ __forceinline__ const V& lanes_at(const float* p, size_t i) { return reinterpret_cast<const V*>(p)[i]; }
+
+template <typename TO, typename V>
+__global__ void __launch_bounds__(256)
+sum_norm_kernel(const SumNormArgs p, TO* __restrict__ rounded) {
+  constexpr int N = Lanes<V>::n;
+  extern __shared__ __align__(16) float row[];
+  __shared__ float scratch[32];
+  pdl_trigger();
+  pdl_wait();
+  const size_t t = blockIdx.x, base = t * p.hidden;
+  const int units = p.hidden / N;
+  float bf[2] = {0.f, 0.f};
+#pragma unroll
+  for (int b = 0; b < 2; ++b) {
+    if (b >= p.branches) continue;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < units; i += blockDim.x) {
+      float f[N];
+      Lanes<V>::get(lanes_at<V>(p.branch[b] + base, i), f);
+#pragma unroll
+      for (int e = 0; e < N; ++e) ss = fmaf(f[e], f[e], ss);
+    }
+    bf[b] = rsqrtf(block_sum(ss, scratch) / static_cast<float>(p.hidden) + p.branch_eps) * p.branch_factor;
+  }
+  const float es = p.extra != nullptr ? p.extra_scale[t] : 0.f;
+  float sum = 0.f;
+  for (int i = threadIdx.x; i < units; i += blockDim.x) {
+    float y[N], f[N], g[N];
+#pragma unroll
+    for (int e = 0; e < N; ++e) y[e] = 0.f;
+    if (p.branches > 0) {
+#pragma unroll
+      for (int b = 0; b < 2; ++b) {
+        if (b >= p.branches) continue;
+        Lanes<V>::get(lanes_at<V>(p.branch[b] + base, i), f);
+        Lanes<V>::get(lanes_at<V>(p.branch_w[b], i), g);
+#pragma unroll
+        for (int e = 0; e < N; ++e) y[e] = fmaf(f[e] * bf[b], g[e], y[e]);
+      }
+    } else if (p.pair_row != nullptr) {
+      for (int j = 0; j < p.top; ++j) {
+        const size_t at = t * p.top + j;
+        const float pw = p.pair_w[at];
+        Lanes<V>::get(lanes_at<V>(p.y + static_cast<size_t>(p.pair_row[at]) * p.hidden, i), f);
+#pragma unroll
+        for (int e = 0; e < N; ++e) y[e] = fmaf(pw, f[e], y[e]);
+      }
+      if (p.extra != nullptr) {
+        Lanes<V>::get(lanes_at<V>(p.extra + base, i), f);
+#pragma unroll
+        for (int e = 0; e < N; ++e) y[e] = fmaf(es, f[e], y[e]);
+      }
+    } else {
+      Lanes<V>::get(lanes_at<V>(p.y + base, i), y);
+    }
+    if (p.s != nullptr) {
+      Lanes<V>::get(lanes_at<V>(p.s, i), g);
+#pragma unroll
+      for (int e = 0; e < N; ++e) y[e] *= g[e];
+    }
+    Lanes<V>::get(lanes_at<V>(p.x + base, i), f);
+#pragma unroll
+    for (int e = 0; e < N; ++e) {
+      f[e] = fmaf(p.alpha, f[e], y[e]);
+      sum += f[e];
+    }
+    reinterpret_cast<V*>(row)[i] = Lanes<V>::put(f);
+  }
+  const float mean = p.centred ? block_sum(sum, scratch) / static_cast<float>(p.hidden) : 0.f;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < units; i += blockDim.x) {
+    float f[N];
+    Lanes<V>::get(lanes_at<V>(row, i), f);
+#pragma unroll
+    for (int e = 0; e < N; ++e) ss = fmaf(f[e] - mean, f[e] - mean, ss);
+  }
+  const float r = rsqrtf(block_sum(ss, scratch) / static_cast<float>(p.hidden) + p.eps);
+  for (int i = threadIdx.x; i < units; i += blockDim.x) {
+    float f[N], g[N];
+    Lanes<V>::get(lanes_at<V>(row, i), f);
+    Lanes<V>::get(lanes_at<V>(p.w, i), g);
+#pragma unroll
+    for (int e = 0; e < N; ++e) f[e] = (f[e] - mean) * r * g[e];
+    reinterpret_cast<V*>(p.x + base)[i] = Lanes<V>::put(f);
+    if (rounded != nullptr) {
+      if constexpr (N == 4) store4(rounded + base + 4 * i, f[0], f[1], f[2], f[3]);
+      else rounded[base + i] = from_float<TO>(f[0]);
+    }
+  }
+}
+
 // out = c0 * z * r1 + c1 * z^2 * r2 + c2 * z^3 * r3 + c3 with r_k = rsqrt(mean over the row of z^(2k) + eps).
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -414,6 +538,28 @@ extern "C" int b200_scale_sum_average(float* x, const float* a, const float* sa,
   else
     launch(scale_sum_average_kernel, dim3(static_cast<unsigned>((total + 255) / 256)), dim3(256), 0, stream, x, a, sa, b, sb, results,
            mix, index, total, C);
+  return launch_status();
+}
+
+extern "C" int b200_sum_norm(float* x, const float* y, const int* pair_row, const float* pair_w, int top, const float* extra,
+                             const float* extra_scale, const float* branch0, const float* branch1, const float* branch_w0,
+                             const float* branch_w1, int branches, float branch_eps, float branch_factor, const float* s,
+                             const float* w, float alpha, float eps, int centred, void* rounded, int n, int hidden, int out_dtype,
+                             cudaStream_t stream) {
+  using namespace b200;
+  if (n <= 0) return 0;
+  if (hidden <= 0 || branches < 0 || branches > 2 || (branches == 0 && y == nullptr) ||
+      (pair_row != nullptr && (pair_w == nullptr || top <= 0)) || (extra != nullptr && (extra_scale == nullptr || pair_row == nullptr)) ||
+      (branches > 0 && (branch0 == nullptr || branch_w0 == nullptr)) || (branches > 1 && (branch1 == nullptr || branch_w1 == nullptr)))
+    return B200_ERR_BAD_SIZE;
+  const size_t smem = sizeof(float) * hidden;
+  if (smem > 48 * 1024) return B200_ERR_TOO_LARGE;
+  const SumNormArgs p{x, y, pair_row, pair_w, top, extra, extra_scale, {branch0, branch1}, {branch_w0, branch_w1}, branches, branch_eps,
+                      branch_factor, s, w, alpha, eps, centred, hidden};
+  const bool vec = hidden % 4 == 0 && aligned16(x, y, extra, branch0, branch1, branch_w0, branch_w1, s, w, rounded);
+  B200_DISPATCH_DTYPE(out_dtype, TO, {
+    launch(vec ? sum_norm_kernel<TO, float4> : sum_norm_kernel<TO, float>, dim3(n), dim3(256), smem, stream, p, static_cast<TO*>(rounded));
+  });
   return launch_status();
 }
 

@@ -791,22 +791,23 @@ __global__ void glu_limit_vec_kernel(const T* __restrict__ gate_up, T* __restric
   *reinterpret_cast<V*>(out + static_cast<size_t>(blockIdx.y) * inter + i) = Vec<T>::pack(y);
 }
 
-// x = cap * tanh(x / cap), element by element, in place (float32)
-__global__ void soft_cap_kernel(float* __restrict__ x, size_t count, float cap) {
+// x = cap * tanh(scale * x / cap), element by element, in place (float32); cap 0: x = scale * x
+__global__ void soft_cap_kernel(float* __restrict__ x, size_t count, float cap, float scale) {
   pdl_trigger();
   pdl_wait();
-  const float inv = 1.f / cap;
+  const float inv = cap > 0.f ? scale / cap : scale;
+  auto capped = [&](float v) { return cap > 0.f ? cap * tanhf(v * inv) : v * inv; };
   const size_t first = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x, stride = static_cast<size_t>(gridDim.x) * blockDim.x;
   const size_t vectors = count / 4;        // the base is on a 16-byte boundary
   for (size_t i = first; i < vectors; i += stride) {
     float4 v = reinterpret_cast<float4*>(x)[i];
-    v.x = cap * tanhf(v.x * inv);
-    v.y = cap * tanhf(v.y * inv);
-    v.z = cap * tanhf(v.z * inv);
-    v.w = cap * tanhf(v.w * inv);
+    v.x = capped(v.x);
+    v.y = capped(v.y);
+    v.z = capped(v.z);
+    v.w = capped(v.w);
     reinterpret_cast<float4*>(x)[i] = v;
   }
-  for (size_t i = vectors * 4 + first; i < count; i += stride) x[i] = cap * tanhf(x[i] * inv);
+  for (size_t i = vectors * 4 + first; i < count; i += stride) x[i] = capped(x[i]);
 }
 
 // out = relu(x)^2, element by element (float32 arithmetic, rounded once)
@@ -924,13 +925,13 @@ extern "C" int b200_glu_limit(const void* gate_up, void* out, int n, int inter, 
   return launch_status();
 }
 
-extern "C" int b200_soft_cap(float* x, long long count, float cap, cudaStream_t stream) {
+extern "C" int b200_soft_cap(float* x, long long count, float cap, float scale, cudaStream_t stream) {
   using namespace b200;
   if (count <= 0) return 0;
-  if (!(cap > 0.f) || (reinterpret_cast<uintptr_t>(x) & 15)) return B200_ERR_BAD_SIZE;
+  if (!(cap >= 0.f) || (reinterpret_cast<uintptr_t>(x) & 15)) return B200_ERR_BAD_SIZE;
   const long long blocks = (count + 1023) / 1024;
   launch(soft_cap_kernel, dim3(static_cast<unsigned>(blocks < 148 * 16 ? blocks : 148 * 16)), dim3(256), 0, stream, x,
-         static_cast<size_t>(count), cap);
+         static_cast<size_t>(count), cap, scale);
   return launch_status();
 }
 

@@ -255,6 +255,9 @@ int launch_grouped_mma(const GroupedArgs& g, int batch, int act, cudaStream_t st
 // score 2: s = softmax(z) over all outputs; the choice goes by s + correction (a float per output, may be null); the outputs
 // form `groups` equal groups of neighbours, a group scores the largest choice score in it, and only outputs of the `keep`
 // best groups can be chosen (the lower index wins a tie, as everywhere); weights = s (without the correction) * scale.
+// score 3: the same with s = sigmoid(z) of every output.  group_best 1: as above; 2: a group scores the sum of the two largest
+// choice scores in it (of the one, where a group is one output).  renorm: the chosen outputs' s are divided by their sum
+// (+ 1e-20) ahead of `scale` (scores 2 and 3).
 // The router's matrix may hold `extra` further rows behind those of the outputs (one number per token each: a gate on
 // something that runs for every token); their logits' sigmoids go to extra_out [n, extra] and take no part in the choice.
 // A CTA takes TOK tokens (batches of many tokens: the router's rows are fetched once for all of them); a token's sums are
@@ -264,7 +267,7 @@ template <typename T, int TOK>
 __global__ void __launch_bounds__(128)
 route_kernel(const T* __restrict__ h, const float* __restrict__ wr, const float* __restrict__ br, int* __restrict__ ids,
              float* __restrict__ wts, int n, int width, int outputs, int top, int score, const float* __restrict__ correction, int groups,
-             int keep, float scale, int extra, float* __restrict__ extra_out) {
+             int keep, float scale, int extra, float* __restrict__ extra_out, int group_best, int renorm) {
   // per token: [experts] logits, [outputs] probabilities, [groups] scores; then [TOK][4][8] partial sums
   extern __shared__ float route_smem[];
   const int experts = outputs + extra;       // rows of the router's matrix
@@ -334,20 +337,23 @@ route_kernel(const T* __restrict__ h, const float* __restrict__ wr, const float*
   float* probs = logits + experts;
   float* group_score = probs + outputs;
   if (lane < extra) extra_out[static_cast<size_t>(token) * extra + lane] = 1.f / (1.f + expf(-logits[outputs + lane]));
-  if (score == 2) {
-    float mx = -INFINITY;
-    for (int e = lane; e < outputs; e += 32) mx = fmaxf(mx, logits[e]);
-    mx = warp_max(mx);
-    float sum = 0.f;
-    for (int e = lane; e < outputs; e += 32) {
-      const float p = expf(logits[e] - mx);
-      probs[e] = p;
-      sum += p;
+  if (score >= 2) {
+    float sum = 1.f;
+    if (score == 2) {
+      float mx = -INFINITY;
+      for (int e = lane; e < outputs; e += 32) mx = fmaxf(mx, logits[e]);
+      mx = warp_max(mx);
+      sum = 0.f;
+      for (int e = lane; e < outputs; e += 32) {
+        const float p = expf(logits[e] - mx);
+        probs[e] = p;
+        sum += p;
+      }
+      sum = warp_sum(sum);
+      __syncwarp();
     }
-    sum = warp_sum(sum);
-    __syncwarp();
     for (int e = lane; e < outputs; e += 32) {
-      const float p = probs[e] / sum;
+      const float p = score == 2 ? probs[e] / sum : 1.f / (1.f + expf(-logits[e]));
       probs[e] = p;
       logits[e] = p + (correction ? correction[e] : 0.f);
     }
@@ -355,9 +361,12 @@ route_kernel(const T* __restrict__ h, const float* __restrict__ wr, const float*
     if (groups > 1) {
       const int per = outputs / groups;
       for (int g = lane; g < groups; g += 32) {
-        float best = -INFINITY;
-        for (int e = g * per; e < (g + 1) * per; ++e) best = fmaxf(best, logits[e]);
-        group_score[g] = best;
+        float best = -INFINITY, second = -INFINITY;
+        for (int e = g * per; e < (g + 1) * per; ++e) {
+          second = fmaxf(second, fminf(best, logits[e]));
+          best = fmaxf(best, logits[e]);
+        }
+        group_score[g] = group_best == 2 && per > 1 ? best + second : best;
       }
       __syncwarp();
       for (int j = 0; j < keep; ++j) {          // the kept groups are marked by +infinity
@@ -405,14 +414,20 @@ route_kernel(const T* __restrict__ h, const float* __restrict__ wr, const float*
     if (lane == 0 && at < outputs) logits[at] = -INFINITY;
     __syncwarp();
   }
+  my_id = min(my_id, outputs - 1);            // nothing left to choose from (every score NaN): still a valid output
+  // the sum of the chosen shares, in the order of the choice (every lane forms the same one)
+  float chosen = 1.f;
+  if (renorm) {
+    chosen = 1e-20f;
+    for (int j = 0; j < top; ++j) chosen += probs[__shfl_sync(0xffffffffu, my_id, j)];
+  }
   if (lane < top) {
-    my_id = min(my_id, outputs - 1);          // nothing left to choose from (every score NaN): still a valid output
     ids[static_cast<size_t>(token) * top + lane] = my_id;
     // score 0: the softmax over the chosen logits; 1: each chosen logit's own sigmoid (the order of sigmoids is the logits');
-    // 2: the chosen output's share of the softmax over all outputs, times scale
+    // 2: the chosen output's share of the softmax over all outputs, times scale; 3: its sigmoid, times scale
     float w = mine / total;
     if (score == 1) w = 1.f / (1.f + expf(-mine_logit));
-    if (score == 2) w = probs[my_id] * scale;
+    if (score >= 2) w = probs[my_id] / chosen * scale;
     wts[static_cast<size_t>(token) * top + lane] = w;
   }
 }
@@ -561,15 +576,16 @@ extern "C" int b200_gemm_grouped(const void* A, long long lda, long long a_z, co
   return B200_ERR_BAD_DTYPE;
 }
 
-// wr float32 [outputs + extra, width]; score 0, 1 or 2 (see route_kernel); correction [outputs] or null; extra_out [n, extra].
+// wr float32 [outputs + extra, width]; score 0 to 3, group_best 1 or 2 (see route_kernel); correction [outputs] or null; extra_out [n, extra].
 extern "C" int b200_moe_route_grouped(const void* h, const float* wr, const float* br, const float* correction, int* ids, float* wts,
                                       float* extra_out, int n, int width, int outputs, int top, int score, int groups, int keep,
-                                      float scale, int extra, int dtype, cudaStream_t stream) {
+                                      float scale, int extra, int group_best, int renorm, int dtype, cudaStream_t stream) {
   using namespace b200;
   if (n <= 0) return 0;
   if (width <= 0 || outputs <= 0 || top <= 0 || top > outputs || top > 32 || outputs > 2048 || extra < 0 || extra > 32 ||
       (extra > 0 && extra_out == nullptr) || groups <= 0 || outputs % groups != 0 || keep <= 0 || keep > groups ||
-      top > keep * (outputs / groups) || score < 0 || score > 2 || (groups > 1 && score != 2))
+      top > keep * (outputs / groups) || score < 0 || score > 3 || (groups > 1 && score < 2) ||
+      (renorm && score < 2) || group_best < 1 || group_best > 2)
     return B200_ERR_BAD_SIZE;
   // many tokens: four a CTA, one choosing warp each (the router's rows cross the L2 a quarter as often)
   const bool four = n >= 512;
@@ -578,9 +594,9 @@ extern "C" int b200_moe_route_grouped(const void* h, const float* wr, const floa
   if (smem > 48 * 1024) return B200_ERR_TOO_LARGE;
   B200_DISPATCH_DTYPE(dtype, T, {
     if (four) launch(route_kernel<T, 4>, dim3((n + 3) / 4), dim3(128), smem, stream, static_cast<const T*>(h), wr, br, ids, wts, n, width,
-                     outputs, top, score, correction, groups, keep, scale, extra, extra_out);
+                     outputs, top, score, correction, groups, keep, scale, extra, extra_out, group_best, renorm);
     else launch(route_kernel<T, 1>, dim3(n), dim3(128), smem, stream, static_cast<const T*>(h), wr, br, ids, wts, n, width, outputs, top,
-                score, correction, groups, keep, scale, extra, extra_out);
+                score, correction, groups, keep, scale, extra, extra_out, group_best, renorm);
   });
   return launch_status();
 }
@@ -588,7 +604,7 @@ extern "C" int b200_moe_route_grouped(const void* h, const float* wr, const floa
 extern "C" int b200_moe_route(const void* h, const float* wr, const float* br, int* ids, float* wts, int n, int width, int experts,
                               int top, int score, int dtype, cudaStream_t stream) {
   if (score < 0 || score > 1) return B200_ERR_BAD_SIZE;
-  return b200_moe_route_grouped(h, wr, br, nullptr, ids, wts, nullptr, n, width, experts, top, score, 1, 1, 1.f, 0, dtype, stream);
+  return b200_moe_route_grouped(h, wr, br, nullptr, ids, wts, nullptr, n, width, experts, top, score, 1, 1, 1.f, 0, 1, 0, dtype, stream);
 }
 
 extern "C" int b200_moe_tile_rows() { return b200::BM; }

@@ -5,18 +5,58 @@
 
 namespace b200 {
 
+// ------------------------------------------------------------- rotation
+// Pair i of the rotated columns is (i, i + half) or, interleaved, (2i, 2i + 1): (u, v) -> (u c - v s, v c + u s) with
+// c = factor * cos(a), s = factor * sin(a), a = p * inv_freq[i].
+struct Rotation {
+  const float* inv_freq;
+  int dims;            // rotated columns, an even number
+  int interleaved;
+  float factor;
+};
+
+// The two columns of pair i.
+__device__ __forceinline__ int pair_first(const Rotation& rot, int i) { return rot.interleaved ? 2 * i : i; }
+__device__ __forceinline__ int pair_second(const Rotation& rot, int i) { return rot.interleaved ? 2 * i + 1 : i + rot.dims / 2; }
+
+// Cosines and sines of one position for all pairs, into shared memory: [dims / 2] cosines, then as many sines.
+__device__ __forceinline__ void rotation_table(float* table, float p, const Rotation& rot) {
+  const int half = rot.dims / 2;
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float sn, cs;
+    sincosf(p * rot.inv_freq[i], &sn, &cs);
+    table[i] = cs * rot.factor;
+    table[half + i] = sn * rot.factor;
+  }
+}
+
+template <typename T>
+__device__ __forceinline__ void rotate_pair(const T* __restrict__ src, T* __restrict__ dst, int i, float p, const Rotation& rot) {
+  float sn, cs;
+  sincosf(p * rot.inv_freq[i], &sn, &cs);
+  sn *= rot.factor;
+  cs *= rot.factor;
+  const int a = pair_first(rot, i), b = pair_second(rot, i);
+  const float u = to_float(src[a]), v = to_float(src[b]);
+  dst[a] = from_float<T>(u * cs - v * sn);
+  dst[b] = from_float<T>(v * cs + u * sn);
+}
+
 // ------------------------------------------------------------- per-head norm and page write
 // Rows [q: nq x d | k: nkv x d | v: nkv x dv | ...].  Each q and k head is divided by its root mean
 // square (eps inside the root), times q_w / k_w (d floats each) where given; q goes to q_out
 // [n, nq, d], k and v into the pages [pages, nkv, page_size, d | dv] at the token's position.
 // `normalise` 0 leaves q and k as they are.  The values start at column v_off of the row: (nq + nkv) * d where v has
-// columns of its own; nq * d where the values are the keys as projected (before their norm; dv = d then).
+// columns of its own; nq * d where the values are the keys as projected (before their norm; dv = d then).  With rotation.dims > 0
+// the first columns of every q and k head are rotated by the token's position behind the norm and its weight.
 template <typename T>
 __global__ void __launch_bounds__(128)
 head_norm_write_kernel(const T* __restrict__ rows, int ld, T* __restrict__ q_out, const float* __restrict__ q_w,
                        const float* __restrict__ k_w, float eps, int normalise, const int* __restrict__ positions,
                        const int* __restrict__ token_entry, const int* __restrict__ block_table, int table_stride,
-                       int page_size, T* __restrict__ k_pool, T* __restrict__ v_pool, int nq, int nkv, int d, int dv, int v_off) {
+                       int page_size, T* __restrict__ k_pool, T* __restrict__ v_pool, int nq, int nkv, int d, int dv, int v_off,
+                       const Rotation rotation) {
+  extern __shared__ float rotated[];        // [rotation.dims]: see rotation_table
   pdl_trigger();
   pdl_wait();
   const int token = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
@@ -24,6 +64,11 @@ head_norm_write_kernel(const T* __restrict__ rows, int ld, T* __restrict__ q_out
   const int p = positions[token];
   const int page = block_table[static_cast<size_t>(token_entry[token]) * table_stride + p / page_size];
   const int in_page = p % page_size;
+  const int half = rotation.dims / 2;
+  if (half > 0) {
+    rotation_table(rotated, static_cast<float>(p), rotation);
+    __syncthreads();
+  }
   for (int head = warp; head < nq + 2 * nkv; head += warps) {
     const bool is_q = head < nq, is_k = !is_q && head < nq + nkv;
     const T* src;
@@ -57,34 +102,24 @@ head_norm_write_kernel(const T* __restrict__ rows, int ld, T* __restrict__ q_out
       }
       f = rsqrtf(warp_sum(ss) / static_cast<float>(width) + eps);
     }
-    for (int i = lane; i < width; i += 32) {
+    const int turned = is_q || is_k ? rotation.dims : 0;
+    for (int i = lane; i < turned / 2; i += 32) {
+      const int a = pair_first(rotation, i), b = pair_second(rotation, i);
+      float u = to_float(src[a]) * f, v = to_float(src[b]) * f;
+      if (w != nullptr) {
+        u *= w[a];
+        v *= w[b];
+      }
+      const float cs = rotated[i], sn = rotated[half + i];
+      dst[a] = from_float<T>(u * cs - v * sn);
+      dst[b] = from_float<T>(v * cs + u * sn);
+    }
+    for (int i = turned + lane; i < width; i += 32) {
       float x = to_float(src[i]) * f;
       if (w != nullptr && (is_q || is_k)) x *= w[i];
       dst[i] = from_float<T>(x);
     }
   }
-}
-
-// ------------------------------------------------------------- rotation
-// Pair i of the rotated columns is (i, i + half) or, interleaved, (2i, 2i + 1): (u, v) -> (u c - v s, v c + u s) with
-// c = factor * cos(a), s = factor * sin(a), a = p * inv_freq[i].
-struct Rotation {
-  const float* inv_freq;
-  int dims;            // rotated columns, an even number
-  int interleaved;
-  float factor;
-};
-
-template <typename T>
-__device__ __forceinline__ void rotate_pair(const T* __restrict__ src, T* __restrict__ dst, int i, float p, const Rotation& rot) {
-  float sn, cs;
-  sincosf(p * rot.inv_freq[i], &sn, &cs);
-  sn *= rot.factor;
-  cs *= rot.factor;
-  const int a = rot.interleaved ? 2 * i : i, b = rot.interleaved ? 2 * i + 1 : i + rot.dims / 2;
-  const float u = to_float(src[a]), v = to_float(src[b]);
-  dst[a] = from_float<T>(u * cs - v * sn);
-  dst[b] = from_float<T>(v * cs + u * sn);
 }
 
 // ------------------------------------------------------------- latent attention: what is kept per token
@@ -151,6 +186,37 @@ rope_slice_kernel(const T* __restrict__ src, int src_ld, int src_head, int src_o
       rotate_pair(s, o, i, p, rotation);
     } else {
       o[rotation.dims + i - half] = s[rotation.dims + i - half];
+    }
+  }
+}
+
+// ------------------------------------------------------------- rotated queries and keys of a recurrence
+// Rows [q: heads x d | k: heads x d | ...] in the storage type -> q_out, k_out float32 [n, heads x d]: the first columns of
+// every head rotated by the token's position, k times k_scale then.  The results are not rounded to the storage type.
+template <typename T>
+__global__ void __launch_bounds__(256)
+rotate_qk_kernel(const T* __restrict__ rows, int ld, float* __restrict__ q_out, float* __restrict__ k_out, int heads, int d,
+                 float k_scale, const Rotation rotation, const int* __restrict__ positions) {
+  extern __shared__ float rotated[];
+  pdl_trigger();
+  pdl_wait();
+  const int token = blockIdx.x, half = rotation.dims / 2, units = half + (d - rotation.dims), all = heads * units;
+  rotation_table(rotated, static_cast<float>(positions[token]), rotation);
+  __syncthreads();
+  for (int j = threadIdx.x; j < 2 * all; j += blockDim.x) {
+    const bool is_k = j >= all;
+    const int r = is_k ? j - all : j, h = r / units, i = r % units;
+    const T* src = rows + static_cast<size_t>(token) * ld + ((is_k ? heads : 0) + h) * d;
+    float* dst = (is_k ? k_out : q_out) + (static_cast<size_t>(token) * heads + h) * d;
+    const float scale = is_k ? k_scale : 1.f;
+    if (i < half) {
+      const int a = pair_first(rotation, i), b = pair_second(rotation, i);
+      const float u = to_float(src[a]), v = to_float(src[b]), cs = rotated[i], sn = rotated[half + i];
+      dst[a] = (u * cs - v * sn) * scale;
+      dst[b] = (v * cs + u * sn) * scale;
+    } else {
+      const int c = rotation.dims + i - half;
+      dst[c] = to_float(src[c]) * scale;
     }
   }
 }
@@ -240,21 +306,31 @@ norm_accumulate_round_kernel(const float* __restrict__ x, const float* __restric
 
 }  // namespace b200
 
-// v_off: the column at which the values' heads start in a row.
+// v_off: the column at which the values' heads start in a row.  rot_dims 0: no rotation.
+extern "C" int b200_head_norm_rotate_write(const void* rows, int ld, void* q_out, const float* q_w, const float* k_w, float eps,
+                                           int normalise, const int* positions, const int* token_entry, const int* block_table,
+                                           int table_stride, int page_size, void* k_pool, void* v_pool, int n, int nq, int nkv, int d,
+                                           int dv, int v_off, int rot_dims, const float* inv_freq, int interleaved, float rot_factor,
+                                           int dtype, cudaStream_t stream) {
+  using namespace b200;
+  if (n <= 0) return 0;
+  if (nq < 0 || nkv < 0 || nq + nkv <= 0 || d <= 0 || dv <= 0 || page_size <= 0 || ld < (nq + nkv) * d || v_off < 0 ||
+      ld < v_off + nkv * dv || rot_dims < 0 || rot_dims % 2 || rot_dims > d || (rot_dims > 0 && inv_freq == nullptr))
+    return B200_ERR_BAD_SIZE;
+  B200_DISPATCH_DTYPE(dtype, T, launch(head_norm_write_kernel<T>, dim3(n), dim3(128), sizeof(float) * rot_dims, stream,
+                                       static_cast<const T*>(rows), ld, static_cast<T*>(q_out), q_w, k_w, eps, normalise, positions,
+                                       token_entry, block_table, table_stride, page_size, static_cast<T*>(k_pool),
+                                       static_cast<T*>(v_pool), nq, nkv, d, dv, v_off,
+                                       Rotation{inv_freq, rot_dims, interleaved, rot_factor}));
+  return launch_status();
+}
+
 extern "C" int b200_head_norm_write_at(const void* rows, int ld, void* q_out, const float* q_w, const float* k_w, float eps,
                                        int normalise, const int* positions, const int* token_entry, const int* block_table,
                                        int table_stride, int page_size, void* k_pool, void* v_pool, int n, int nq, int nkv, int d,
                                        int dv, int v_off, int dtype, cudaStream_t stream) {
-  using namespace b200;
-  if (n <= 0) return 0;
-  if (nq < 0 || nkv < 0 || nq + nkv <= 0 || d <= 0 || dv <= 0 || page_size <= 0 || ld < (nq + nkv) * d || v_off < 0 ||
-      ld < v_off + nkv * dv)
-    return B200_ERR_BAD_SIZE;
-  B200_DISPATCH_DTYPE(dtype, T, launch(head_norm_write_kernel<T>, dim3(n), dim3(128), 0, stream, static_cast<const T*>(rows), ld,
-                                       static_cast<T*>(q_out), q_w, k_w, eps, normalise, positions, token_entry, block_table,
-                                       table_stride, page_size, static_cast<T*>(k_pool), static_cast<T*>(v_pool), nq, nkv, d, dv,
-                                       v_off));
-  return launch_status();
+  return b200_head_norm_rotate_write(rows, ld, q_out, q_w, k_w, eps, normalise, positions, token_entry, block_table, table_stride,
+                                     page_size, k_pool, v_pool, n, nq, nkv, d, dv, v_off, 0, nullptr, 0, 1.f, dtype, stream);
 }
 
 extern "C" int b200_head_norm_write(const void* rows, int ld, void* q_out, const float* q_w, const float* k_w, float eps,
@@ -263,6 +339,19 @@ extern "C" int b200_head_norm_write(const void* rows, int ld, void* q_out, const
                                     int dv, int dtype, cudaStream_t stream) {
   return b200_head_norm_write_at(rows, ld, q_out, q_w, k_w, eps, normalise, positions, token_entry, block_table, table_stride,
                                  page_size, k_pool, v_pool, n, nq, nkv, d, dv, (nq + nkv) * d, dtype, stream);
+}
+
+extern "C" int b200_rotate_qk(const void* rows, int ld, float* q_out, float* k_out, int n, int heads, int d, float k_scale,
+                              int rot_dims, const float* inv_freq, int interleaved, float rot_factor, const int* positions, int dtype,
+                              cudaStream_t stream) {
+  using namespace b200;
+  if (n <= 0) return 0;
+  if (heads <= 0 || d <= 0 || 2 * heads * d > ld || rot_dims < 0 || rot_dims % 2 || rot_dims > d || (rot_dims > 0 && inv_freq == nullptr))
+    return B200_ERR_BAD_SIZE;
+  B200_DISPATCH_DTYPE(dtype, T, launch(rotate_qk_kernel<T>, dim3(n), dim3(256), sizeof(float) * rot_dims, stream,
+                                       static_cast<const T*>(rows), ld, q_out, k_out, heads, d, k_scale,
+                                       Rotation{inv_freq, rot_dims, interleaved, rot_factor}, positions));
+  return launch_status();
 }
 
 extern "C" int b200_latent_prepare(const void* rows, int ld, int q_off, int q_rank, const float* q_w, void* cq_out, int kv_off,

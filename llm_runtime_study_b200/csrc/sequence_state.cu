@@ -3,11 +3,11 @@
 //   linear scan     S_t = D_t S_(t-1) + k_t u_t^T,  o_t = S_t^T q_t        per head, S is [d, dv]
 //                   (the delta rule's read-out is formed as (D_t S_(t-1))^T q_t + u_t (k_t . q_t), the same sum)
 //                   D_t = one decay per head (a constant), a diagonal of per-row factors g_t (gated), or one factor per
-//                         row and head (row gates)
+//                         row and head (row gates; token gates, which carry no normaliser)
 //                   u_t = v_t (plain), beta_t (v_t - (D_t S_(t-1))^T k_t) (delta rule), or b_t v_t (row gates, which also
 //                         carry n_t = D_t n_(t-1) + b_t k_t and give n_t . q_t: the matrix memory's normaliser)
 //   short convolution over time per channel, with the last taps-1 inputs kept per request
-//   per-group RMS norm of the read-out times a sigmoid or SiLU gate
+//   per-group RMS norm of the read-out (with or without a weight) times a sigmoid or SiLU gate
 //   the gates themselves: exponential input and forget gates kept in range by a running maximum, decays per key channel
 //                   from a low-rank map
 //
@@ -42,12 +42,12 @@ struct ScanParams {
   float* out; int ldo;                            // [n, H * dv]
   const int* q_start; const int* slots;           // per entry: first token, request slot
   int H, Hqk, d, dv, act, rl;                     // act 1: silu on q, k, v as they are read; rl: lanes that share a column
-  const float* row_decay; const float* row_gain;  // [n, H]: D_t and b_t (row gates)
+  const float* row_decay; const float* row_gain;  // [n, H]: D_t (row and token gates) and b_t (row gates)
   float* norm_state; float* norm_out;             // [slots, H, d], [n, H]: n and n . q (row gates)
   float q_scale;                                  // on q as it is read
 };
 
-enum ScanGate : int { GATE_HEAD = 0, GATE_CHANNEL = 1, GATE_ROW = 2 };
+enum ScanGate : int { GATE_HEAD = 0, GATE_CHANNEL = 1, GATE_ROW = 2, GATE_TOKEN = 3 };
 
 constexpr int kScanThreads = 128;
 // tokens staged in shared memory at a time: 16, or 8 where a token's rows are more than 128 wide
@@ -63,13 +63,14 @@ constexpr int scan_chunk(int dpt, int rl) { return dpt * rl <= 128 ? 16 : 8; }
 // what a launch with few requests and long portions wants: its time is a chain of dependent steps,
 // and the chain per token is a quarter as long.
 // GATE_ROW: the normaliser n is one more column of the state, behind the last value column, whose value is 1 for every
-// token; it lives in an array of its own.
-template <typename T, int DPT, int RL, bool DELTA, int GATE>
+// token; it lives in an array of its own.  TV: the storage type of v, where q and k come in another one (float32 rows that a
+// kernel ahead has prepared).
+template <typename T, typename TV, int DPT, int RL, bool DELTA, int GATE>
 __global__ void __launch_bounds__(kScanThreads) linear_scan_kernel(const ScanParams p) {
   extern __shared__ __align__(16) float smem[];
   pdl_trigger();
   pdl_wait();
-  constexpr bool GATED = GATE == GATE_CHANNEL, ROW = GATE == GATE_ROW;
+  constexpr bool GATED = GATE == GATE_CHANNEL, ROW = GATE == GATE_ROW, TOKEN = ROW || GATE == GATE_TOKEN;
   static_assert(!(DELTA && ROW), "row gates and the delta rule exclude each other");
   constexpr int rl = RL, cols_per_warp = 32 / rl, cols = (kScanThreads / 32) * cols_per_warp;
   constexpr int dp = DPT * rl;                          // rows padded to dp >= d; the padding holds zeros
@@ -99,16 +100,17 @@ __global__ void __launch_bounds__(kScanThreads) linear_scan_kernel(const ScanPar
   float* gs = qs + CHUNK * dp;                   // [chunk][dp] (gated only)
   float* vs = gs + (GATED ? CHUNK * dp : 0);     // [chunk][cols]
   float* bs = vs + CHUNK * cols;                 // [chunk]: beta (delta rule) or b (row gates)
-  float* ds = bs + CHUNK;                        // [chunk]: the head's factor of the token (row gates)
+  float* ds = bs + CHUNK;                        // [chunk]: the head's factor of the token (row and token gates)
   float dec = GATE == GATE_HEAD ? p.decay[h] : 1.f;
   const T* qg = static_cast<const T*>(p.q);
   const T* kg = static_cast<const T*>(p.k);
-  const T* vg = static_cast<const T*>(p.v);
+  const TV* vg = static_cast<const TV*>(p.v);
 
   // The rows of the next chunk are asked for before the tokens of this one are worked through, and land in
   // registers; they go to shared memory (SiLU applied once per element) when this chunk is done.
   // (kept in the storage type: a conversion right behind the load would wait for it)
-  T rk[EPT], rq[EPT], rv[VPT];
+  T rk[EPT], rq[EPT];
+  TV rv[VPT];
   float rg[EPT], rb = 0.f, rd = 0.f;
   auto fetch = [&](int t0, int count) {
 #pragma unroll
@@ -130,13 +132,11 @@ __global__ void __launch_bounds__(kScanThreads) linear_scan_kernel(const ScanPar
       if (e * kScanThreads >= count * cols) break;
       const int idx = threadIdx.x + e * kScanThreads;
       const int tt = idx / cols, c = cb * cols + idx % cols;
-      rv[e] = (tt < count && c < dv) ? vg[static_cast<size_t>(t0 + tt) * p.ldv + h * dv + c] : from_float<T>(ROW && c == dv ? 1.f : 0.f);
+      rv[e] = (tt < count && c < dv) ? vg[static_cast<size_t>(t0 + tt) * p.ldv + h * dv + c] : from_float<TV>(ROW && c == dv ? 1.f : 0.f);
     }
     if (DELTA && threadIdx.x < count) rb = p.beta[static_cast<size_t>(t0 + threadIdx.x) * p.ldb + h];
-    if (ROW && threadIdx.x < count) {
-      rb = p.row_gain[static_cast<size_t>(t0 + threadIdx.x) * p.H + h];
-      rd = p.row_decay[static_cast<size_t>(t0 + threadIdx.x) * p.H + h];
-    }
+    if (ROW && threadIdx.x < count) rb = p.row_gain[static_cast<size_t>(t0 + threadIdx.x) * p.H + h];
+    if (TOKEN && threadIdx.x < count) rd = p.row_decay[static_cast<size_t>(t0 + threadIdx.x) * p.H + h];
   };
   auto stash = [&](int count) {
 #pragma unroll
@@ -151,10 +151,10 @@ __global__ void __launch_bounds__(kScanThreads) linear_scan_kernel(const ScanPar
     for (int e = 0; e < VPT; ++e) {
       if (e * kScanThreads >= count * cols) break;
       const int idx = threadIdx.x + e * kScanThreads;
-      if (idx < CHUNK * cols) vs[idx] = p.act ? silu_of<T>(to_float(rv[e])) : to_float(rv[e]);
+      if (idx < CHUNK * cols) vs[idx] = p.act ? silu_of<TV>(to_float(rv[e])) : to_float(rv[e]);
     }
     if ((DELTA || ROW) && threadIdx.x < CHUNK) bs[threadIdx.x] = rb;
-    if (ROW && threadIdx.x < CHUNK) ds[threadIdx.x] = rd;
+    if (TOKEN && threadIdx.x < CHUNK) ds[threadIdx.x] = rd;
   };
 
   fetch(t_begin, min(CHUNK, t_end - t_begin));
@@ -177,6 +177,7 @@ __global__ void __launch_bounds__(kScanThreads) linear_scan_kernel(const ScanPar
       const float4* gt = reinterpret_cast<const float4*>(gs + tt * dp + r * DPT);
       float4 kk[DPT / 4];
       float o_sum;
+      if (TOKEN) dec = ds[tt];
       if constexpr (DELTA) {
         // o = (D S)^T q + u (k . q): the three sums over rows (against k, against q, and k . q) are formed in one
         // pass and reduced over the lanes together, so a token costs one shuffle tree, not two in a row
@@ -222,7 +223,6 @@ __global__ void __launch_bounds__(kScanThreads) linear_scan_kernel(const ScanPar
         }
       } else {
         const float u = ROW ? vs[tt * cols + col_local] * bs[tt] : vs[tt * cols + col_local];
-        if (ROW) dec = ds[tt];
         float acc[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
         for (int v = 0; v < DPT / 4; ++v) {
@@ -260,7 +260,7 @@ __global__ void __launch_bounds__(kScanThreads) linear_scan_kernel(const ScanPar
   }
 }
 
-template <typename T, bool DELTA, int GATE>
+template <typename T, typename TV, bool DELTA, int GATE>
 int launch_scan(ScanParams p, int entries, cudaStream_t stream) {
   const int dpt = (p.d + p.rl - 1) / p.rl;
   const int cols = (kScanThreads / 32) * (32 / p.rl);
@@ -274,7 +274,7 @@ int launch_scan(ScanParams p, int entries, cudaStream_t stream) {
   if (smem > 48 * 1024) return B200_ERR_TOO_LARGE;
 #define B200_SCAN_CASE(DPT_, RL_)                                                                                      \
   if (dpt8 == DPT_ && p.rl == RL_) {                                                                                   \
-    launch(linear_scan_kernel<T, DPT_, RL_, DELTA, GATE>, grid, dim3(kScanThreads), smem, stream, p);                 \
+    launch(linear_scan_kernel<T, TV, DPT_, RL_, DELTA, GATE>, grid, dim3(kScanThreads), smem, stream, p);                 \
     return launch_status();                                                                                            \
   }
   B200_SCAN_CASE(8, 4) B200_SCAN_CASE(16, 4) B200_SCAN_CASE(24, 4) B200_SCAN_CASE(32, 4)
@@ -305,9 +305,9 @@ struct DeltaPrepareParams {
   const float* taps; int ntaps;    // [C, ntaps], C = 2 G d + H dv channels in the order q, k, v
   const float* conv_state;         // [slots, ntaps - 1, C]: inputs of the positions before this step, oldest first
   const float* a_log;              // [H]
-  const float* dt_bias;            // [H d]
+  const float* dt_bias;            // [H d], or [H] (rank 0)
   const void* a_up;                // [rank, H d] storage type (the map's weight transposed: neighbouring threads read neighbouring outputs)
-  float* q; float* k; float* v; float* g; float* beta;   // [n, G d], [n, G d], [n, H dv], [n, H d], [n, H]
+  float* q; float* k; float* v; float* g; float* beta;   // [n, G d], [n, G d], [n, H dv], [n, H d] or [n, H] (rank 0), [n, H]
   const int* q_start; const int* slots; const int* token_entry;
   int H, G, d, dv;
   float unit_eps, q_scale;
@@ -317,8 +317,8 @@ struct DeltaPrepareParams {
 // heads x tokens CTAs; more for prompt portions, so that the head's taps and its slice of the low-rank map are
 // fetched once per CTA into shared memory).  Per token: the convolution and SiLU of the head's value channels, of its
 // q and k channels (the first head of a group of heads that share them does these), their unit norms, the head's
-// decay factors g = exp(-exp(a_log) * softplus(low-rank(x) + dt_bias)), and beta = sigmoid(.).  Every sum has an
-// order that depends on the sizes only.
+// decay factors g = exp(-exp(a_log) * softplus(low-rank(x) + dt_bias)), and beta = sigmoid(.).  rank 0: no low-rank map; the
+// head has one decay a token, its logit at column a_off + h.  Every sum has an order that depends on the sizes only.
 template <typename T>
 __global__ void __launch_bounds__(128) delta_prepare_kernel(const DeltaPrepareParams p, int n, int tokens_per_cta) {
   extern __shared__ float smem[];
@@ -382,6 +382,13 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const DeltaPreparePa
     }
     __syncthreads();             // low[] is complete
     if (threadIdx.x == 0) p.beta[static_cast<size_t>(t) * p.H + h] = sigmoid_f(to_float(proj[static_cast<size_t>(t) * p.ld + p.b_off + h]));
+    if (p.rank == 0) {
+      if (threadIdx.x == 32) {
+        const float a = to_float(proj[static_cast<size_t>(t) * p.ld + p.a_off + h]);
+        p.g[static_cast<size_t>(t) * p.H + h] = expf(-rate * softplus_f(a + p.dt_bias[h]));
+      }
+      continue;
+    }
     for (int i = threadIdx.x; i < d; i += blockDim.x) {
       const size_t col = static_cast<size_t>(h) * d + i;
       float a = 0.f;
@@ -514,7 +521,8 @@ __global__ void conv_state_update_kernel(const T* __restrict__ proj, int ld, flo
 // ------------------------------------------------------------- group norm times sigmoid gate
 // out[t, c] = y[t, c] * rsqrt(mean over c's group of y^2 + eps) * w[c % w_len] * act(gate[t, c]), act the sigmoid or SiLU;
 // y = x, or, with `den` and `floor` ([n, width / group] each), y = x / (max(|den|, floor) + den_eps) with its group's two
-// numbers.  w_len is the group's size (one weight for all groups) or the width.  The gate's logits are read from `gate_in` directly (rank 0) or formed as gate_up[:, c] . gate_in[t, :rank]
+// numbers.  w_len is the group's size (one weight for all groups) or the width; w may be null (no weight).
+// The gate's logits are read from `gate_in` directly (rank 0) or formed as gate_up[:, c] . gate_in[t, :rank]
 // (gate_up is [rank, width]: the map's weight transposed).
 template <typename T>
 __global__ void group_norm_gate_kernel(const float* __restrict__ x, int width, int group, const float* __restrict__ w, int w_len,
@@ -547,7 +555,7 @@ __global__ void group_norm_gate_kernel(const float* __restrict__ x, int width, i
       logit = 0.f;
       for (int j = 0; j < rank; ++j) logit = fmaf(to_float(gate_up[static_cast<size_t>(j) * width + c]), low[j], logit);
     }
-    out[static_cast<size_t>(t) * width + c] = from_float<T>(row[i] * f * wg[i] * (gate_silu ? silu_f(logit) : sigmoid_f(logit)));
+    out[static_cast<size_t>(t) * width + c] = from_float<T>(row[i] * f * (w != nullptr ? wg[i] : 1.f) * (gate_silu ? silu_f(logit) : sigmoid_f(logit)));
   }
 }
 
@@ -556,26 +564,37 @@ __global__ void group_norm_gate_kernel(const float* __restrict__ x, int width, i
 // `tokens`: rows in the batch (with `entries` it tells a batch of single tokens from one that holds portions).
 // `fixed_order`: the same lanes per column whatever the batch looks like, so that a token's bits do not depend on the cut.
 // q, k: [n, Hqk * d] rows (strides ldq, ldk), v: [n, H * dv]; element type by `dtype`.  gate (float32 [n, H * d]) selects
-// per-row factors, else `decay` ([H]) is used; beta (float32 [n, H]) selects the delta rule.  state float32 [slots, H, d, dv].
+// per-row factors, row_decay (float32 [n, H]) one factor per row and head (the delta rule only), else `decay` ([H]) is used; beta
+// (float32 [n, H]) selects the delta rule.  state float32 [slots, H, d, dv].  v_dtype: v's element type, another one than q's and
+// k's with a constant decay and without the delta rule only.
 extern "C" int b200_linear_scan(const void* q, const void* k, const void* v, int ldq, int ldk, int ldv, const float* gate, int ldg,
-                                const float* decay, const float* beta, int ldb, float* state, float* out, int ldo,
+                                const float* decay, const float* row_decay, const float* beta, int ldb, float* state, float* out, int ldo,
                                 const int* q_start, const int* slots, int entries, int tokens, int H, int Hqk, int d, int dv,
-                                int act, float q_scale, int fixed_order, int dtype, cudaStream_t stream) {
+                                int act, float q_scale, int fixed_order, int dtype, int v_dtype, cudaStream_t stream) {
   using namespace b200;
   if (entries <= 0) return 0;
   if (H <= 0 || Hqk <= 0 || H % Hqk != 0 || d <= 0 || dv <= 0 || d > 256) return B200_ERR_BAD_SIZE;
-  if ((gate == nullptr) == (decay == nullptr)) return B200_ERR_BAD_SIZE;
-  ScanParams p{q, k, v, ldq, ldk, ldv, gate, ldg, decay, beta, ldb, state, out, ldo, q_start, slots, H, Hqk, d, dv, act, 1, nullptr, nullptr, nullptr, nullptr, q_scale};
+  if ((gate != nullptr) + (decay != nullptr) + (row_decay != nullptr) != 1) return B200_ERR_BAD_SIZE;
+  ScanParams p{q, k, v, ldq, ldk, ldv, gate, ldg, decay, beta, ldb, state, out, ldo, q_start, slots, H, Hqk, d, dv, act, 1, row_decay, nullptr, nullptr, nullptr, q_scale};
   p.rl = scan_row_lanes(entries, H, d, dv, tokens, fixed_order);
   const bool delta = beta != nullptr, gated = gate != nullptr;
+  if (v_dtype != dtype) {
+    if (delta || decay == nullptr || dtype != kF32 || v_dtype != kBF16) return B200_ERR_BAD_DTYPE;
+    return launch_scan<float, __nv_bfloat16, false, GATE_HEAD>(p, entries, stream);
+  }
+  if (row_decay != nullptr) {
+    if (!delta) return B200_ERR_BAD_SIZE;
+    if (dtype != kF32) return B200_ERR_BAD_DTYPE;        // what delta_prepare writes
+    return launch_scan<float, float, true, GATE_TOKEN>(p, entries, stream);
+  }
   if (delta && gated) {
-    B200_DISPATCH_DTYPE(dtype, T, return (launch_scan<T, true, GATE_CHANNEL>(p, entries, stream)));
+    B200_DISPATCH_DTYPE(dtype, T, return (launch_scan<T, T, true, GATE_CHANNEL>(p, entries, stream)));
   } else if (!delta && !gated) {
-    B200_DISPATCH_DTYPE(dtype, T, return (launch_scan<T, false, GATE_HEAD>(p, entries, stream)));
+    B200_DISPATCH_DTYPE(dtype, T, return (launch_scan<T, T, false, GATE_HEAD>(p, entries, stream)));
   } else if (delta) {
-    B200_DISPATCH_DTYPE(dtype, T, return (launch_scan<T, true, GATE_HEAD>(p, entries, stream)));
+    B200_DISPATCH_DTYPE(dtype, T, return (launch_scan<T, T, true, GATE_HEAD>(p, entries, stream)));
   } else {
-    B200_DISPATCH_DTYPE(dtype, T, return (launch_scan<T, false, GATE_CHANNEL>(p, entries, stream)));
+    B200_DISPATCH_DTYPE(dtype, T, return (launch_scan<T, T, false, GATE_CHANNEL>(p, entries, stream)));
   }
   return 0;
 }
@@ -592,7 +611,7 @@ extern "C" int b200_linear_scan_row_gates(const void* q, const void* k, const vo
   ScanParams p{q, k, v, ldq, ldk, ldv, nullptr, 0, nullptr, nullptr, 0, state, out, H * dv, q_start, slots, H, H, d, dv, 0, 1,
                decay, gain, norm_state, norm_out, q_scale};
   p.rl = scan_row_lanes(entries, H, d, dv + 1, tokens, fixed_order);
-  B200_DISPATCH_DTYPE(dtype, T, return (launch_scan<T, false, GATE_ROW>(p, entries, stream)));
+  B200_DISPATCH_DTYPE(dtype, T, return (launch_scan<T, T, false, GATE_ROW>(p, entries, stream)));
   return 0;
 }
 
@@ -671,7 +690,7 @@ extern "C" int b200_group_norm_gate(const float* x, int n, int width, int group,
                                     const void* gate_up, int gate_silu, void* out, int dtype, cudaStream_t stream) {
   using namespace b200;
   if (n <= 0) return 0;
-  if (width <= 0 || group <= 0 || width % group != 0 || rank < 0 || rank > 4096 || (w_len != group && w_len != width) ||
+  if (width <= 0 || group <= 0 || width % group != 0 || rank < 0 || rank > 4096 || (w != nullptr && w_len != group && w_len != width) ||
       (den == nullptr) != (floor_ == nullptr))
     return B200_ERR_BAD_SIZE;
   dim3 grid(n, width / group);

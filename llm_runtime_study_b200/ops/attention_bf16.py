@@ -20,6 +20,7 @@ _MIN_KEYS_PER_SPLIT = 128
 
 _TABLE = {
     "b200_attention_head_dim": [],
+    "b200_attention_value_dim": [],
     "b200_attention_prefill_rows": [],
     "b200_attention_prefill_bf16": [c_void_p] * 6 + [c_int, c_int, c_int, c_int, c_float, c_int] + [c_void_p] * 3 + [c_int, c_void_p],
     "b200_attention_decode_scratch_floats": [c_int, c_int, c_int],
@@ -113,15 +114,29 @@ def tma_supported(head_dim: int, page_size: int, window: int) -> bool:
     return head_dim % 64 == 0 and head_dim <= MAX_HEAD_DIM and page_size % 16 == 0 and not window
 
 
-def library_name(head_dim: int) -> str:
-    name = f"b200_attention_mma_d{head_dim}"
+def library_name(head_dim: int, value_dim: int | None = None) -> str:
+    """The mma.sync library of a head size (``value_dim``: of the values, where it is another one)."""
+
+    if value_dim in (None, head_dim):
+        name, defines = f"b200_attention_mma_d{head_dim}", (f"HEAD_DIM={head_dim}",)
+    else:
+        name, defines = f"b200_attention_mma_d{head_dim}_v{value_dim}", (f"HEAD_DIM={head_dim}", f"VALUE_DIM={value_dim}")
     if name not in native.library_specs():
-        native.register_library(name, ("attention_mma.cu",), _TABLE, defines=(f"HEAD_DIM={head_dim}",))
+        native.register_library(name, ("attention_mma.cu",), _TABLE, defines=defines)
     return name
 
 
 def supported(head_dim: int) -> bool:
     return head_dim % 16 == 0 and 16 <= head_dim <= MAX_HEAD_DIM
+
+
+def build_pair(head_dim: int, value_dim: int) -> None:
+    """Compile the mma.sync kernels for keys and values of different head sizes."""
+
+    from ..csrc.build import build_library
+
+    name = library_name(head_dim, value_dim)
+    build_library(name, ("attention_mma.cu",), native.library_defines(name))
 
 
 def build(head_dim: int) -> None:

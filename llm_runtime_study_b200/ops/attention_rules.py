@@ -16,10 +16,13 @@ BACKEND = os.environ.get("LLM_RUNTIME_STUDY_B200_ATTENTION_RULES", "tcgen05")
 
 
 def tensor_core_supported(q: torch.Tensor, cache: Any) -> bool:
-    """bfloat16, keys and values of one head size that the mma.sync kernels are built for."""
+    """bfloat16, keys and values of head sizes that the mma.sync kernels can be built for."""
 
-    d = q.shape[2]
-    return (q.dtype == torch.bfloat16 and cache.values.shape[3] == d and attention_bf16.supported(d))
+    return q.dtype == torch.bfloat16 and attention_bf16.supported(q.shape[2]) and attention_bf16.supported(cache.values.shape[3])
+
+
+def _output(q: torch.Tensor, values: torch.Tensor) -> torch.Tensor:
+    return torch.empty((*q.shape[:2], values.shape[3]), dtype=q.dtype, device=q.device)
 
 
 def paged_attention_rules(q: torch.Tensor, cache: Any, ctx: Any, table: torch.Tensor, *, scale: float, window: int = 0,
@@ -30,7 +33,7 @@ def paged_attention_rules(q: torch.Tensor, cache: Any, ctx: Any, table: torch.Te
     the sink's ``1 +`` in the denominator, and a mask in blocks (``chunk > 0``: a position sees its own block of ``chunk``
     positions, counted from 0, only).
 
-    float32 runtime, and shapes no tensor-core kernel takes (values of another head size than the keys): the
+    float32 runtime, and shapes no tensor-core kernel takes (head sizes that are no multiple of 16): the
     CUDA-core kernel (one warp per token and head, float32 arithmetic, tiles of 32 keys from key 0, so the order
     of every sum depends on the token's position alone).  bfloat16 runtime: the kernels of the plain attention,
     built a second time with the rules applied to the score tile: for batches that hold prompt portions the tcgen05
@@ -44,10 +47,12 @@ def paged_attention_rules(q: torch.Tensor, cache: Any, ctx: Any, table: torch.Te
         n, nq, d = q.shape
         keys, values = cache.keys, cache.values
         _, _, _, nkv, page_size, gs, slices = attention_bf16._geometry(q, keys)
-        lib = attention_bf16.library_name(d)
-        out = torch.empty_like(q)
+        dv = values.shape[3]
+        lib = attention_bf16.library_name(d, dv)
+        out = _output(q, values)
         if ctx.all_decode and n == ctx.num_entries:
-            splits = attention_bf16.decode_splits(n, nkv, slices, ctx.max_kv_len, head_dim=d)
+            reach = min(ctx.max_kv_len, window) if window else ctx.max_kv_len
+            splits = attention_bf16.decode_splits(n, nkv, slices, reach, head_dim=(d + dv) // 2)
             floats = native.query("b200_attention_decode_scratch_floats", n, nq, splits, library=lib)
             scratch = torch.empty(max(floats, 1), dtype=torch.float32, device=q.device)
             native.call(
@@ -57,7 +62,7 @@ def paged_attention_rules(q: torch.Tensor, cache: Any, ctx: Any, table: torch.Te
                 library=lib, launches=2 if splits > 1 else 1)
             return out
         maps = ctx.__dict__.setdefault("_tile_maps", {})
-        if (BACKEND == "tcgen05" and attention_bf16.PREFILL_BACKEND == "tcgen05" and attention_bf16.tc_supported(d, page_size, window)
+        if (BACKEND == "tcgen05" and attention_bf16.PREFILL_BACKEND == "tcgen05" and dv == d and attention_bf16.tc_supported(d, page_size, window)
                 and ctx.max_q_len >= attention_bf16.TC_MIN_PORTION):
             per_tile = 128 // gs
             key = ("tc", per_tile)
@@ -97,11 +102,12 @@ def _masked(q: torch.Tensor, cache: Any, ctx: Any, table: torch.Tensor, *, scale
         n, nq, d = q.shape
         keys, values = cache.keys, cache.values
         _, _, _, nkv, page_size, gs, slices = attention_bf16._geometry(q, keys)
-        lib = attention_bf16.library_name(d)
-        out = torch.empty_like(q)
+        dv = values.shape[3]
+        lib = attention_bf16.library_name(d, dv)
+        out = _output(q, values)
         if ctx.all_decode and n == ctx.num_entries:
             reach = min(ctx.max_kv_len, chunk) if chunk else ctx.max_kv_len
-            splits = attention_bf16.decode_splits(n, nkv, slices, reach, head_dim=d)
+            splits = attention_bf16.decode_splits(n, nkv, slices, reach, head_dim=(d + dv) // 2)
             floats = native.query("b200_attention_decode_scratch_floats", n, nq, splits, library=lib)
             scratch = torch.empty(max(floats, 1), dtype=torch.float32, device=q.device)
             native.call(

@@ -1,5 +1,5 @@
 """Kernels of a layer whose sublayers read one normalised copy of the stream side by side: layer norm, the short
-convolution added to each sublayer's input, the scaled sum of the sublayers' outputs with the average over all layers'
+convolution added to each sublayer's input, the norm of a scaled stream plus a sublayer's output, the scaled sum of the sublayers' outputs with the average over all layers'
 results, the polynomial activation of normalised powers, and the gated unit of rows whose router weight multiplies the
 expert's input.  Statistics and sums are float32 in both run types."""
 
@@ -8,6 +8,7 @@ from __future__ import annotations
 import torch
 
 from ..errors import KernelError
+from .mixer_steps import NormedBranches, PairedRows
 from .native import call, ptr, require, stream_ptr, tag
 
 
@@ -78,6 +79,52 @@ def scale_sum_average(x: torch.Tensor, a: torch.Tensor, scale_a: torch.Tensor | 
             raise KernelError(f"results have shape {tuple(results.shape)}, expected [>= {index + 2}, {n}, {width}]")
     call("b200_scale_sum_average", ptr(x), ptr(a), ptr(scale_a), ptr(b), ptr(scale_b), ptr(results) if mix is not None else None,
          ptr(mix), index, n, width, stream_ptr())
+
+
+def sum_norm(x: torch.Tensor, y: "torch.Tensor | PairedRows | NormedBranches", weight: torch.Tensor, eps: float, *, alpha: float,
+             scale: torch.Tensor | None = None, centred: bool = True, rounded_dtype: torch.dtype | None = None) -> torch.Tensor | None:
+    """In place on the float32 stream ``x`` ``[N, C]``: ``x <- norm(alpha * x + scale * y) * weight`` with the layer norm
+    (``centred``) or the RMS norm; ``scale`` is one factor per column.  ``y`` may be ``PairedRows`` or ``NormedBranches``: the sublayer's
+    output is then formed inside the kernel.  With ``rounded_dtype`` the new rows are also returned in that type.  The width is at
+    most 12,288 (a row is kept in shared memory)."""
+
+    require(x, "x", dtype=torch.float32, dims=2)
+    n, width = x.shape
+    require(weight, "weight", dtype=torch.float32, shape=(width,))
+    if scale is not None:
+        require(scale, "scale", dtype=torch.float32, shape=(width,))
+    rows = pair_row = pair_w = extra = extra_scale = None
+    top = 0
+    branches: list = []
+    branch_w: list = []
+    branch_eps, factor = 0.0, 1.0
+    if isinstance(y, NormedBranches):
+        branches, branch_w, branch_eps, factor = list(y.rows), list(y.weights), y.eps, y.factor
+        if not 0 < len(branches) <= 2 or len(branch_w) != len(branches):
+            raise KernelError("sum_norm takes one or two branches with a weight each")
+        for b, w in zip(branches, branch_w):
+            require(b, "branch", dtype=torch.float32, shape=x.shape)
+            require(w, "branch weight", dtype=torch.float32, shape=(width,))
+    elif isinstance(y, PairedRows):
+        rows, pair_row, pair_w, extra, extra_scale = y.rows, y.pair_row, y.weights, y.extra, y.extra_scale
+        top = pair_w.shape[1]
+        require(rows, "rows", dtype=torch.float32, dims=2)
+        if rows.shape[1] != width or pair_w.shape[0] != n:
+            raise KernelError("sum_norm: the paired rows do not fit the stream")
+        if extra is not None:
+            require(extra, "extra", dtype=torch.float32, shape=x.shape)
+            require(extra_scale, "extra_scale", dtype=torch.float32)
+            if extra_scale.numel() != n:
+                raise KernelError("sum_norm: one factor per token is expected")
+    else:
+        rows = require(y, "y", dtype=torch.float32, shape=x.shape)
+    rounded = None if rounded_dtype is None else torch.empty((n, width), dtype=rounded_dtype, device=x.device)
+    b = branches + [None] * (2 - len(branches))
+    w = branch_w + [None] * (2 - len(branch_w))
+    call("b200_sum_norm", ptr(x), ptr(rows), ptr(pair_row), ptr(pair_w), top, ptr(extra), ptr(extra_scale), ptr(b[0]), ptr(b[1]),
+         ptr(w[0]), ptr(w[1]), len(branches), float(branch_eps), float(factor), ptr(scale), ptr(weight), float(alpha), float(eps),
+         1 if centred else 0, ptr(rounded), n, width, tag(rounded_dtype or torch.float32), stream_ptr())
+    return rounded
 
 
 def poly_norm(z: torch.Tensor, coef: torch.Tensor, eps: float) -> torch.Tensor:

@@ -262,11 +262,11 @@ def relu2(x: torch.Tensor) -> torch.Tensor:
     return out
 
 
-def soft_cap(x: torch.Tensor, cap: float) -> torch.Tensor:
-    """``x <- cap * tanh(x / cap)`` in place on float32 values; ``x`` is returned."""
+def soft_cap(x: torch.Tensor, cap: float | None, scale: float = 1.0) -> torch.Tensor:
+    """``x <- cap * tanh(scale * x / cap)`` (``cap`` ``None``: ``scale * x``) in place on float32 values; ``x`` is returned."""
 
     require(x, "x", dtype=torch.float32)
-    call("b200_soft_cap", ptr(x), x.numel(), float(cap), stream_ptr())
+    call("b200_soft_cap", ptr(x), x.numel(), float(cap or 0.0), float(scale), stream_ptr())
     return x
 
 

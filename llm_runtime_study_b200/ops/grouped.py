@@ -79,17 +79,19 @@ def tile_rows() -> int:
     return query("b200_moe_tile_rows")
 
 
-SCORES = {"softmax_chosen": 0, "sigmoid": 1, "softmax_all": 2}
+SCORES = {"softmax_chosen": 0, "sigmoid": 1, "softmax_all": 2, "sigmoid_all": 3}
 
 
 def route(h: torch.Tensor, router: torch.Tensor, bias: torch.Tensor | None, *, top: int, wide_tiles: bool = False,
           score: str = "softmax_chosen", correction: torch.Tensor | None = None, groups: int = 1, keep: int = 1,
-          scale: float = 1.0, identity: int = 0, extra: int = 0) -> Routing:
+          scale: float = 1.0, identity: int = 0, extra: int = 0, group_best: int = 1, renormalise: bool = False) -> Routing:
     """Logits ``router @ h + bias`` in float32 (``router`` float32 ``[outputs + extra, width]``; ``h`` in the activation type), the
     ``top`` largest chosen (the lower index wins a tie); weights by ``score``: the softmax over the chosen logits, each chosen
     logit's sigmoid (not renormalised), or (``softmax_all``) the chosen outputs' shares ``s`` of the softmax over all outputs
     times ``scale``, where the choice goes by ``s + correction`` among the outputs of the ``keep`` best of ``groups`` equal
-    groups of neighbours (a group scores its largest choice score).  The last ``identity`` outputs have no expert behind them
+    groups of neighbours (a group scores its largest choice score, or the sum of its ``group_best`` = 2 largest); ``sigmoid_all``: the
+    same with ``s`` the sigmoid of every output's logit.  ``renormalise``: the chosen outputs' ``s`` are divided by their sum
+    (+ 1e-20) ahead of ``scale``.  The last ``identity`` outputs have no expert behind them
     (their pairs get no row: ``pair_row`` -1).  ``extra`` further rows of ``router`` give one number per token each, whose
     sigmoids are returned in ``Routing.extra``.  Then the pairs sorted by expert, each expert's rows padded to whole tiles
     (of 128 rows with ``wide_tiles``, what the tcgen05 kernel takes; else of 64)."""
@@ -114,7 +116,8 @@ def route(h: torch.Tensor, router: torch.Tensor, bias: torch.Tensor | None, *, t
     if score not in SCORES:
         raise KernelError(f"unknown router score {score!r}; expected one of {sorted(SCORES)}")
     call("b200_moe_route_grouped", ptr(h), ptr(router), ptr(bias), ptr(correction), ptr(ids), ptr(weights), ptr(extra_out), n, width,
-         outputs, top, SCORES[score], int(groups), int(keep), float(scale), int(extra), tag(h.dtype), stream_ptr())
+         outputs, top, SCORES[score], int(groups), int(keep), float(scale), int(extra), int(group_best), 1 if renormalise else 0,
+         tag(h.dtype), stream_ptr())
     tile = TC_TILE_ROWS if wide_tiles else tile_rows()
     max_tiles = min(-(-n * top // tile) + experts, n * top)       # a tile holds one expert's rows only
     pair_row = torch.empty(n * top, dtype=torch.int32, device=dev)

@@ -17,12 +17,25 @@ from .native import call, ptr, query, require, stream_ptr, tag
 @dataclass
 class PairedRows:
     """A sublayer's output given in pieces: row ``t`` is ``sum_j weights[t, j] * rows[pair_row[t * top + j]]`` (what the experts a
-    router chose returned for token ``t``).  A consumer that reads the rows anyway forms the sum itself."""
+    router chose returned for token ``t``), plus ``extra_scale[t] * extra[t]`` where given (what runs for every token).  A consumer
+    that reads the rows anyway forms the sum itself."""
 
     rows: torch.Tensor          # float32 [sorted rows, width]
     pair_row: torch.Tensor      # int32 [N * top]
     weights: torch.Tensor       # float32 [N, top]
+    extra: torch.Tensor | None = None           # float32 [N, width]
+    extra_scale: torch.Tensor | None = None     # float32, one number per token
 
+
+@dataclass
+class NormedBranches:
+    """A sublayer's output given as its branches: ``factor * sum_b rows_b * rsqrt(mean(rows_b^2) + eps) * weight_b`` (one or two
+    branches).  A consumer that reads the rows anyway forms it itself."""
+
+    rows: "list[torch.Tensor]"          # float32 [N, width] each
+    weights: "list[torch.Tensor]"       # float32 [width] each
+    eps: float
+    factor: float
 
 
 def head_norm_write(
@@ -30,11 +43,13 @@ def head_norm_write(
     q_weight: torch.Tensor | None = None, k_weight: torch.Tensor | None = None, normalise: bool = True,
     positions: torch.Tensor, token_entry: torch.Tensor, block_table: torch.Tensor, page_size: int,
     k_pool: torch.Tensor, v_pool: torch.Tensor, value_offset: int | None = None,
+    rotary: "tuple[torch.Tensor, int, bool, float] | None" = None,
 ) -> torch.Tensor:
     """Rows ``[q | k | v | ...]``: every q and k head divided by its root mean square (``eps`` inside the root), times a
     weight of ``head_dim`` floats where given; q is returned ``[N, nq, d]``, k and v go into the pages
     ``[pages, nkv, page_size, d | dv]`` at each token's position.  ``value_offset``: the column at which the values' heads
-    start (default: behind the keys); ``nq * d`` makes the values the keys as projected, before their norm."""
+    start (default: behind the keys); ``nq * d`` makes the values the keys as projected, before their norm.  ``rotary = (inv_freq,
+    rotated columns, interleaved, factor)``: q and k are rotated by the position behind the norm (see ``latent_prepare``)."""
 
     require(rows, "rows", dims=2)
     n, ld = rows.shape
@@ -55,10 +70,39 @@ def head_norm_write(
         raise KernelError(f"pools have shapes {tuple(k_pool.shape)} and {tuple(v_pool.shape)}, expected "
                           f"[pages, {num_kv_heads}, {page_size}, {head_dim} | {value_dim}]")
     q_out = torch.empty((n, num_q_heads, head_dim), dtype=dt, device=rows.device)
-    call("b200_head_norm_write_at", ptr(rows), ld, ptr(q_out), ptr(q_weight), ptr(k_weight), float(eps), 1 if normalise else 0,
+    inv_freq, rot_dims, interleaved, factor = _rotary(rotary, head_dim)
+    call("b200_head_norm_rotate_write", ptr(rows), ld, ptr(q_out), ptr(q_weight), ptr(k_weight), float(eps), 1 if normalise else 0,
          ptr(positions), ptr(token_entry), ptr(block_table), block_table.shape[1], page_size, ptr(k_pool), ptr(v_pool), n,
-         num_q_heads, num_kv_heads, head_dim, value_dim, int(value_offset), tag(dt), stream_ptr())
+         num_q_heads, num_kv_heads, head_dim, value_dim, int(value_offset), rot_dims, ptr(inv_freq), 1 if interleaved else 0,
+         float(factor), tag(dt), stream_ptr())
     return q_out
+
+
+def _rotary(rotary: "tuple[torch.Tensor, int, bool, float] | None", head_dim: int):
+    if rotary is None:
+        return None, 0, False, 1.0
+    inv_freq, rot_dims, interleaved, factor = rotary
+    if rot_dims % 2 or not 0 < rot_dims <= head_dim:
+        raise KernelError(f"{rot_dims} rotated columns do not fit heads of {head_dim}")
+    require(inv_freq, "inv_freq", dtype=torch.float32, shape=(rot_dims // 2,))
+    return inv_freq, rot_dims, interleaved, factor
+
+
+def rotate_qk(rows: torch.Tensor, *, heads: int, head_dim: int, positions: torch.Tensor,
+              rotary: "tuple[torch.Tensor, int, bool, float] | None", k_scale: float = 1.0) -> tuple[torch.Tensor, torch.Tensor]:
+    """Rows ``[q | k | ...]`` (``heads`` heads of ``head_dim`` each): both rotated by the token's position (``rotary`` as for
+    ``head_norm_write``), k times ``k_scale`` then; float32 ``[N, heads * head_dim]`` each, not rounded to the rows' type."""
+
+    require(rows, "rows", dims=2)
+    n, ld = rows.shape
+    if ld < 2 * heads * head_dim:
+        raise KernelError(f"rows of width {ld} do not hold q and k of {heads} heads of {head_dim}")
+    require(positions, "positions", dtype=torch.int32, shape=(n,))
+    inv_freq, rot_dims, interleaved, factor = _rotary(rotary, head_dim)
+    q, k = torch.empty((2, n, heads * head_dim), dtype=torch.float32, device=rows.device)
+    call("b200_rotate_qk", ptr(rows), ld, ptr(q), ptr(k), n, heads, head_dim, float(k_scale), rot_dims, ptr(inv_freq),
+         1 if interleaved else 0, float(factor), ptr(positions), tag(rows.dtype), stream_ptr())
+    return q, k
 
 
 def latent_prepare(
@@ -140,6 +184,8 @@ def norm_accumulate_round(x: "torch.Tensor | PairedRows | None", weight: torch.T
     pair_row = pair_w = None
     top = 0
     if isinstance(x, PairedRows):
+        if x.extra is not None:
+            raise KernelError("norm_accumulate_round forms the sum over a token's pairs only")
         pair_row, pair_w, top, x = x.pair_row, x.weights, x.weights.shape[1], x.rows
         require(x, "rows", dtype=torch.float32, dims=2)
         if x.shape[1] != hidden or pair_w.shape[0] != n:

@@ -52,7 +52,7 @@ _LIBRARIES = {
             "b200_rmsnorm_accumulate": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_int, c_void_p],
             "b200_add_rows": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
             "b200_relu2": [c_void_p, c_void_p, c_longlong, c_int, c_void_p],
-            "b200_soft_cap": [c_void_p, c_longlong, c_float, c_void_p],
+            "b200_soft_cap": [c_void_p, c_longlong, c_float, c_float, c_void_p],
         },
     ),
     "b200_embedding_sum": (
@@ -98,8 +98,8 @@ _LIBRARIES = {
         ("sequence_state.cu",),
         {
             "b200_linear_scan": [
-                c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p,
-                c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p,
+                c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
+                c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_void_p,
             ],
             "b200_linear_scan_row_gates": [
                 c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
@@ -125,6 +125,11 @@ _LIBRARIES = {
                                      c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
             "b200_head_norm_write_at": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_int, c_void_p, c_void_p, c_void_p,
                                         c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+            "b200_head_norm_rotate_write": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_int, c_void_p, c_void_p, c_void_p,
+                                            c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
+                                            c_int, c_float, c_int, c_void_p],
+            "b200_rotate_qk": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_float,
+                               c_void_p, c_int, c_void_p],
             "b200_latent_prepare": [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int,
                                     c_void_p, c_int, c_float, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int,
                                     c_void_p],
@@ -152,7 +157,7 @@ _LIBRARIES = {
                                   c_int, c_int, c_int, c_void_p],
             "b200_moe_route": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
             "b200_moe_route_grouped": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                                       c_int, c_int, c_int, c_float, c_int, c_int, c_void_p],
+                                       c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_int, c_void_p],
             "b200_moe_combine_mixed": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                        c_void_p],
             "b200_moe_tile_rows": [],
@@ -169,6 +174,8 @@ _LIBRARIES = {
                                c_int, c_int, c_int, c_void_p],
             "b200_scale_sum_average": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                                        c_void_p],
+            "b200_sum_norm": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                              c_int, c_float, c_float, c_void_p, c_void_p, c_float, c_float, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
             "b200_poly_norm": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_void_p],
             "b200_silu_mul_scaled": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
         },

@@ -10,6 +10,7 @@ import torch
 from ..ops import attention_bf16
 from ..ops import attention_rules
 from ..ops import functional as F
+from ..ops import mixer_steps as M
 from ..weights.checkpoint import TensorSpec
 from ..weights.view import TensorView
 from .base import MIXERS, NORMS, POSITION_ENCODINGS, Mixer, PagedKV, PagedTensors, Runtime
@@ -235,4 +236,80 @@ class SinkAttention(Mixer):
             q, cache, ctx, table, scale=self.scale, window=self.window or 0, softcap=self.softcap or 0.0,
             slopes=self.slopes, sink=self.sink,
         )
+        return self.o_proj(out.view(out.shape[0], -1), torch.float32)
+
+
+@MIXERS.register("capped_attention")
+class CappedAttention(Mixer):
+    """Grouped-query causal attention with capped scores: ``q = W_q x``, ``k = W_k x`` (heads of ``head_dim``), ``v = W_v x`` (heads of
+    ``value_dim``), no biases.  Every q and k head is RMS-normed with one weight of ``head_dim`` numbers for all heads (``q.norm``,
+    ``k.norm``; ``qk_norm_eps`` inside the root; ``None``: no norm), then rotated by the position (``position``: a rotary encoding over
+    the leading columns, in either layout and with a factor; ``None``: no rotation).  ``S = scale * q.k``; ``S <- softcap * tanh(S /
+    softcap)`` (``None``: no cap); position i sees j with ``0 <= i - j < window`` (``None``: all before it); ordinary softmax; ``W_o``.
+    Query head h reads key/value head ``h // (heads / kv_heads)``.  Tensors: ``q``, ``k``, ``v`` (one stacked product), ``q.norm``,
+    ``k.norm``, ``o``.  The pages hold the rotated keys."""
+
+    graph_safe = True
+
+    def __init__(self, *, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int, value_dim: int | None = None,
+                 scale: float | None = None, qk_norm_eps: float | None = None, softcap: float | None = None, window: int | None = None,
+                 position: Mapping[str, Any] | None = None) -> None:
+        value_dim = head_dim if value_dim is None else value_dim
+        if min(hidden_size, num_heads, num_kv_heads, head_dim, value_dim) <= 0:
+            raise ValueError("attention sizes must be positive")
+        if num_heads % num_kv_heads:
+            raise ValueError(f"num_heads {num_heads} is not a multiple of num_kv_heads {num_kv_heads}")
+        if head_dim > 256 or value_dim > 256:
+            raise ValueError(f"head sizes {head_dim} and {value_dim} must be at most 256: no kernel takes larger ones")
+        if (softcap is not None and softcap <= 0) or (window is not None and window <= 0):
+            raise ValueError("a soft cap and a window must be positive")
+        self.hidden_size, self.num_heads, self.num_kv_heads = hidden_size, num_heads, num_kv_heads
+        self.head_dim, self.value_dim = head_dim, value_dim
+        self.scale = 1.0 / math.sqrt(head_dim) if scale is None else float(scale)
+        self.qk_norm_eps = None if qk_norm_eps is None else float(qk_norm_eps)
+        self.softcap, self.window = None if softcap is None else float(softcap), window
+        self.position = POSITION_ENCODINGS.build(position) if position else None
+
+    def children(self):
+        return (self.position,) if self.position is not None else ()
+
+    def tensor_specs(self) -> dict[str, TensorSpec]:
+        h, d = self.hidden_size, self.head_dim
+        specs = {
+            "q": TensorSpec((self.num_heads * d, h)), "k": TensorSpec((self.num_kv_heads * d, h)),
+            "v": TensorSpec((self.num_kv_heads * self.value_dim, h)), "o": TensorSpec((h, self.num_heads * self.value_dim)),
+        }
+        if self.qk_norm_eps is not None:
+            specs["q.norm"] = TensorSpec((d,), init="one_plus_normal", std=0.05)
+            specs["k.norm"] = TensorSpec((d,), init="one_plus_normal", std=0.05)
+        return specs
+
+    def load(self, tensors: Mapping[str, torch.Tensor], runtime: Runtime) -> None:
+        self.runtime = runtime
+        self.qkv_proj = Projection([tensors["q"], tensors["k"], tensors["v"]], None, runtime)
+        self.o_proj = Projection([tensors["o"]], None, runtime)
+        self.q_weight = self.k_weight = None
+        if self.qk_norm_eps is not None:
+            self.q_weight = runtime.place_vector_f32(tensors["q.norm"])
+            self.k_weight = runtime.place_vector_f32(tensors["k.norm"])
+        if self.position is not None:
+            self.position.load({}, runtime)
+
+    def cache_requirement(self) -> PagedTensors:
+        return PagedTensors(
+            tensors=(("keys", (self.num_kv_heads, self.head_dim)), ("values", (self.num_kv_heads, self.value_dim))),
+            window=self.window,
+        )
+
+    def forward(self, x: torch.Tensor, ctx: Any, cache: Any) -> torch.Tensor:
+        qkv = self.qkv_proj(x)
+        table = ctx.block_table(cache.group)
+        q = M.head_norm_write(
+            qkv, num_q_heads=self.num_heads, num_kv_heads=self.num_kv_heads, head_dim=self.head_dim, value_dim=self.value_dim,
+            eps=self.qk_norm_eps or 0.0, q_weight=self.q_weight, k_weight=self.k_weight, normalise=self.qk_norm_eps is not None,
+            positions=ctx.positions, token_entry=ctx.token_entry, block_table=table, page_size=cache.page_size, k_pool=cache.keys,
+            v_pool=cache.values, rotary=self.position.rotary_layout() if self.position is not None else None,
+        )
+        out = attention_rules.paged_attention_rules(q, cache, ctx, table, scale=self.scale, window=self.window or 0,
+                                                    softcap=self.softcap or 0.0)
         return self.o_proj(out.view(out.shape[0], -1), torch.float32)

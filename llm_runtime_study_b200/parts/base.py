@@ -139,6 +139,13 @@ class Norm(Part):
 
         return None
 
+    def row_norm(self) -> tuple[torch.Tensor, float, bool] | None:
+        """(weight, eps, centred) if the norm is ``weight * (x - m) * rsqrt(mean((x - m)^2) + eps)`` with ``m`` the row's mean
+        (``centred``) or 0; ``None`` for any other norm."""
+
+        fusable = self.fusable()
+        return None if fusable is None else (*fusable, False)
+
     def add_norm(self, resid: torch.Tensor, delta: torch.Tensor | None) -> torch.Tensor:
         raise NotImplementedError
 

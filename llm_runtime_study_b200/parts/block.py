@@ -143,6 +143,77 @@ class OutputNormBlock(Block):
             stream.rounded = x
 
 
+@BLOCKS.register("sum_norm")
+class SumNormBlock(Block):
+    """``h = norm_1(alpha h + s1 * mixer(h)); h = norm_2(alpha h + s2 * ffn(h))``: the norm sits behind the sum, so the rows the
+    sublayers read (rounded to the activation type where that is not float32) are normed already.  ``layer_scale``: ``s1`` and ``s2``
+    are vectors of the width (otherwise 1).  One kernel forms the sum, norms it into the float32 rows and hands the next sublayer
+    its rounded copy; it also forms a sublayer's output from its pieces (branches of a parallel mixer, a router's experts and a
+    gated shared one) where the sublayer can hand them over.  ``names`` as for ``pre_norm``, with ``mixer_scale`` and ``ffn_scale``; a
+    layer without a feed-forward is its first half only."""
+
+    graph_safe = True
+
+    def __init__(
+        self, *, hidden_size: int, mixer: Mapping[str, Any], feed_forward: Mapping[str, Any] | None, mixer_norm: Mapping[str, Any],
+        ffn_norm: Mapping[str, Any] | None = None, names: Mapping[str, str] | None = None, alpha: float = 1.0, layer_scale: bool = False,
+    ) -> None:
+        self.hidden_size, self.alpha, self.layer_scale = hidden_size, float(alpha), bool(layer_scale)
+        self.names = {**_DEFAULT_NAMES, "mixer_scale": "ls1", "ffn_scale": "ls2", **(names or {})}
+        self.mixer = MIXERS.build(mixer)
+        self.mixer_norm = NORMS.build(mixer_norm)
+        self.feed_forward = FEED_FORWARDS.build(feed_forward) if feed_forward else None
+        self.ffn_norm = NORMS.build(ffn_norm) if feed_forward else None
+        if feed_forward and not ffn_norm:
+            raise ValueError("a sum_norm block with a feed-forward needs the norm behind it (ffn_norm)")
+        for norm in (self.mixer_norm, self.ffn_norm):
+            if norm is not None and norm.row_norm() is None:
+                raise ValueError("a sum_norm block takes a layer norm or an RMS norm")
+
+    def children(self):
+        return tuple(part for _, part in self._parts())
+
+    _parts = PreNormBlock._parts
+
+    def _scales(self) -> tuple[str, ...]:
+        if not self.layer_scale:
+            return ()
+        return ("mixer_scale", "ffn_scale") if self.feed_forward is not None else ("mixer_scale",)
+
+    def tensor_specs(self) -> dict[str, TensorSpec]:
+        specs = {f"{prefix}.{n}": s for prefix, part in self._parts() for n, s in part.tensor_specs().items()}
+        specs.update({self.names[s]: TensorSpec((self.hidden_size,), init="one_plus_normal", std=0.2) for s in self._scales()})
+        return specs
+
+    def load(self, tensors: Mapping[str, torch.Tensor], runtime: Runtime) -> None:
+        PreNormBlock.load(self, tensors, runtime)
+        self.scales = {s: runtime.place_vector_f32(tensors[self.names[s]]) for s in self._scales()}
+
+    def forward(self, stream: ResidualStream, ctx: Any, cache: Any) -> None:
+        from ..ops import block_steps as B
+        from ..ops import mixer_steps as M
+
+        resid, act = stream.resid, self.runtime.dtype
+        if stream.delta is not None:
+            resid += stream.delta
+        rounded = act if act != torch.float32 else None
+        x = stream.rounded          # what the block before this one left for its reader, if it made such a copy
+        stream.put(None, None)
+        if x is None:
+            x = resid if rounded is None else M.norm_accumulate_round(None, None, 0.0, resid, act)
+        steps = [(self.mixer, (ctx, cache), self.mixer_norm, "mixer_scale")]
+        if self.feed_forward is not None:
+            steps.append((self.feed_forward, (ctx,), self.ffn_norm, "ffn_scale"))
+        for part, args, norm, scale in steps:
+            whole = getattr(part, "returns_pieces", False) or getattr(part, "returns_gated_pieces", False)
+            out = part.forward(x, *args, **({"pieces": True} if whole else {}))
+            weight, eps, centred = norm.row_norm()
+            x = B.sum_norm(resid, out, weight, eps, alpha=self.alpha, scale=self.scales.get(scale), centred=centred, rounded_dtype=rounded)
+            if rounded is None:
+                x = resid
+        stream.rounded = x if rounded is not None else None
+
+
 _PARALLEL_NAMES = {
     "norm": "norm1", "mixer": "mix", "feed_forward": "mlp", "mixer_scale": "ls1", "ffn_scale": "ls2",
     "mixer_taps": "canon1", "ffn_taps": "canon2", "average": "dwa",

@@ -117,18 +117,19 @@ class SummedEmbedding(Part):
 
 @HEADS.register("linear_head")
 class OutputHead(Part):
-    """``logits = h W^T`` in float32, no bias (mini_llm/model/qwen.py:112), with ``softcap``
+    """``logits = scale * h W^T`` in float32, no bias (mini_llm/model/qwen.py:112; ``scale`` 1), with ``softcap``
     ``softcap * tanh(logits / softcap)`` of them.  With
     ``tied`` the weight may be absent from the checkpoint; the embedding matrix
     is used then.  A stored ``lm_head.weight`` is always used when present."""
 
     graph_safe = True
 
-    def __init__(self, *, vocab_size: int, hidden_size: int, tied: bool = False, softcap: float | None = None) -> None:
+    def __init__(self, *, vocab_size: int, hidden_size: int, tied: bool = False, softcap: float | None = None,
+                 scale: float = 1.0) -> None:
         if softcap is not None and softcap <= 0:
             raise ValueError("a soft cap must be positive")
         self.vocab_size, self.hidden_size, self.tied = vocab_size, hidden_size, bool(tied)
-        self.softcap = None if softcap is None else float(softcap)
+        self.softcap, self.scale = None if softcap is None else float(softcap), float(scale)
 
     def tensor_specs(self) -> dict[str, TensorSpec]:
         return {"weight": TensorSpec((self.vocab_size, self.hidden_size), optional=self.tied)}
@@ -148,4 +149,4 @@ class OutputHead(Part):
 
     def forward(self, x: "torch.Tensor | WeightedRows") -> torch.Tensor:
         logits = self.proj(x, torch.float32)
-        return logits if self.softcap is None else F.soft_cap(logits, self.softcap)
+        return logits if self.softcap is None and self.scale == 1.0 else F.soft_cap(logits, self.softcap, self.scale)

@@ -28,7 +28,9 @@ class RoutedExperts(FeedForward):
     * ``score``: ``softmax_chosen``: the weights are the softmax over the chosen logits only; ``sigmoid``: each chosen
       expert's ``sigmoid(z)``, not renormalised; ``softmax_all``: ``s = softmax(z)`` over all router outputs, the choice goes
       by ``s + correction`` (``correction``: a stored vector) among the outputs of the ``keep`` best of ``groups`` equal groups of
-      neighbours (a group scores its largest choice score), the weights are ``weight_scale * s`` of the chosen, not renormalised.
+      neighbours (a group scores its largest choice score, or the sum of its ``group_best`` = 2 largest), the weights are
+      ``weight_scale * s`` of the chosen, not renormalised; ``sigmoid_all``: the same with ``s = sigmoid(z)`` of every output.  With
+      ``renormalise`` the chosen outputs' ``s`` are divided by their sum (+ 1e-20) first.
     * ``identity``: that many further router outputs behind the experts' that have no tensors and return their input.
     * ``weight_on``: ``output``: the result is ``sum w_e expert_e(x)``; ``input``: ``sum expert_e(w_e x)``.
     * ``shared_size``: a further expert of that inner size (same form; ``shared_limit``) that runs for every token and is
@@ -48,7 +50,7 @@ class RoutedExperts(FeedForward):
                  router_bias: bool = True, score: str = "softmax_chosen", weight_on: str = "output",
                  shared_size: int | None = None, limit: float | None = None, alpha: float = 1.702, correction: bool = False,
                  groups: int = 1, keep: int = 1, weight_scale: float = 1.0, identity: int = 0, shared_limit: float | None = None,
-                 shared_gate: bool = False) -> None:
+                 shared_gate: bool = False, group_best: int = 1, renormalise: bool = False) -> None:
         if min(hidden_size, intermediate_size, experts, top) <= 0 or top > experts:
             raise ValueError("expert sizes must be positive and top at most the number of experts")
         if act not in ACTS:
@@ -66,8 +68,10 @@ class RoutedExperts(FeedForward):
         outputs = experts + identity
         if identity < 0 or groups <= 0 or outputs % groups or not 0 < keep <= groups or top > keep * (outputs // groups):
             raise ValueError("router outputs must form equal groups, and the kept groups must hold at least `top` outputs")
-        if (groups > 1 or correction or identity or weight_scale != 1.0) and score != "softmax_all":
-            raise ValueError("groups, a correction, identity outputs and a weight scale belong to the score 'softmax_all'")
+        if (groups > 1 or correction or identity or weight_scale != 1.0 or renormalise) and score not in ("softmax_all", "sigmoid_all"):
+            raise ValueError("groups, a correction, identity outputs, a weight scale and renormalised weights belong to the scores over all outputs")
+        if group_best not in (1, 2):
+            raise ValueError(f"a group scores its largest choice score or the sum of its two largest, got group_best {group_best}")
         if identity and weight_on != "output":
             raise ValueError("identity outputs are weighted on the output")
         if shared_gate and shared_size is None:
@@ -75,6 +79,7 @@ class RoutedExperts(FeedForward):
         self.hidden_size, self.intermediate_size, self.experts, self.top = hidden_size, intermediate_size, experts, top
         self.act, self.router_bias, self.score, self.weight_on, self.shared_size = act, bool(router_bias), score, weight_on, shared_size
         self.limit, self.alpha, self.correction, self.groups, self.keep = limit, float(alpha), bool(correction), groups, keep
+        self.group_best, self.renormalise = int(group_best), bool(renormalise)
         self.weight_scale, self.identity, self.shared_limit, self.shared_gate = float(weight_scale), identity, shared_limit, bool(shared_gate)
 
     def tensor_specs(self) -> dict[str, TensorSpec]:
@@ -123,6 +128,11 @@ class RoutedExperts(FeedForward):
     def returns_pieces(self) -> bool:
         return self.shared_size is None and self.weight_on == "output" and not self.identity
 
+    # the same with the gated shared expert's rows and their factors beside them (``PairedRows.extra``)
+    @property
+    def returns_gated_pieces(self) -> bool:
+        return self.shared_gate and self.weight_on == "output" and not self.identity
+
     def forward(self, x: torch.Tensor, ctx: Any, *, pieces: bool = False) -> "torch.Tensor | PairedRows":
         """``pieces``: return the experts' rows with the pairing instead of their weighted sum, for a consumer that forms the
         sum while it reads the rows anyway (the norm behind this part does)."""
@@ -130,7 +140,7 @@ class RoutedExperts(FeedForward):
         wide = G.wide_tiles_pay(x.shape[0], self.top, x.dtype, self.hidden_size, self.intermediate_size)
         routing = G.route(x, self.router, self.router_b, top=self.top, wide_tiles=wide, score=self.score, correction=self.correction_b,
                           groups=self.groups, keep=self.keep, scale=self.weight_scale, identity=self.identity,
-                          extra=1 if self.shared_gate else 0)
+                          extra=1 if self.shared_gate else 0, group_best=self.group_best, renormalise=self.renormalise)
         if self.act == "limited_glu":
             on_input = False
             hidden = F.glu_limit(G.expert_linear(x, self.up, routing, gather=True), self.limit, self.alpha)
@@ -144,6 +154,8 @@ class RoutedExperts(FeedForward):
         rows = G.expert_linear(hidden, self.down, routing, gather=False, out_dtype=torch.float32)
         if pieces and self.returns_pieces:
             return PairedRows(rows, routing.pair_row, routing.weights)
+        if pieces and self.returns_gated_pieces:
+            return PairedRows(rows, routing.pair_row, routing.weights, self.shared_down(self._shared_hidden(x), torch.float32), routing.extra)
         if self.identity or self.shared_gate:
             # one pass forms the weighted sum, hands an identity output the token's own row, and adds the gated shared expert
             shared = self.shared_down(self._shared_hidden(x), torch.float32) if self.shared_gate else None

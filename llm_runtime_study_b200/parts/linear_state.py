@@ -7,10 +7,11 @@ from typing import Any, Mapping, Sequence
 import torch
 
 from ..ops import functional as F
+from ..ops import mixer_steps as M
 from ..ops import sequence_state as S
 from ..weights.checkpoint import TensorSpec
 from ..weights.view import TensorView
-from .base import MIXERS, FixedState, Mixer, PagedTensors, Runtime
+from .base import MIXERS, POSITION_ENCODINGS, FixedState, Mixer, PagedTensors, Runtime
 from .linear import Projection
 
 
@@ -74,56 +75,71 @@ class DecayedLinearAttention(Mixer):
 
 @MIXERS.register("gated_delta_rule")
 class GatedDeltaRule(Mixer):
-    """The delta rule with one decay per head and key channel.  ``q``, ``k`` (``qk_heads x dim``) and ``v``
+    """The delta rule with one decay per head and key channel, or per head.  ``q``, ``k`` (``qk_heads x dim``) and ``v``
     (``heads x vdim``) each pass a causal convolution over time per channel (``taps`` taps, the last one the
     current token's, zeros before the start) and SiLU; q and k become unit vectors per head
     (``x / sqrt(sum x^2 + unit_eps)``), q also times ``dim^(-1/2)``.  ``beta = sigmoid(W_b x)`` per head;
-    ``g = exp(-exp(A_log_h) * softplus(W_a2 (W_a1 x) + dt_bias))`` per head and key channel.  Per head, in this
+    ``g = exp(-exp(A_log_h) * softplus(W_a2 (W_a1 x) + dt_bias))`` per head and key channel, or, with ``decay_rank`` ``None``,
+    ``g = exp(-exp(A_log_h) * softplus(W_a x + dt_bias))`` per head.  Per head, in this
     order: ``S <- diag(g) S``, ``u = beta (v - S^T k)``, ``S <- S + k u^T``, ``o = S^T q``.  Each head's ``o`` is
     divided by its root mean square, times ``norm`` (``vdim``, shared by the heads), times
-    ``sigmoid(W_g2 (W_g1 x))``, then ``W_o``.  Head ``h`` reads q/k head ``h // (heads / qk_heads)``.
+    ``act(W_g2 (W_g1 x))`` or, with ``gate_rank`` ``None``, ``act(W_g x)`` (``gate_act``: sigmoid or silu), then ``W_o``.  Head ``h``
+    reads q/k head ``h // (heads / qk_heads)``.
 
     Per request: the float32 state ``[heads, dim, vdim]`` and the last ``taps - 1`` inputs of the convolutions.
-    Tensors: ``q``, ``k``, ``v``, ``b``, ``a1``, ``g1`` (one stacked product), ``q.conv``, ``k.conv``, ``v.conv``,
-    ``A_log``, ``dt_bias``, ``a2``, ``g2``, ``norm``, ``o``."""
+    Tensors: ``q``, ``k``, ``v``, ``b``, ``a1`` or ``a``, ``g1`` or ``g`` (one stacked product), ``q.conv``, ``k.conv``,
+    ``v.conv``, ``A_log``, ``dt_bias``, ``a2``, ``g2``, ``norm``, ``o``."""
 
     graph_safe = True
 
     def __init__(self, *, hidden_size: int, num_heads: int, num_qk_heads: int, head_dim: int, value_dim: int, taps: int,
-                 decay_rank: int, gate_rank: int, eps: float, unit_eps: float = 1e-6) -> None:
-        if min(hidden_size, num_heads, num_qk_heads, head_dim, value_dim, taps, decay_rank, gate_rank) <= 0 or head_dim > 256:
+                 decay_rank: int | None, gate_rank: int | None, eps: float, unit_eps: float = 1e-6, gate_act: str = "sigmoid") -> None:
+        ranks = [rank for rank in (decay_rank, gate_rank) if rank is not None]
+        if min(hidden_size, num_heads, num_qk_heads, head_dim, value_dim, taps, *ranks) <= 0 or head_dim > 256:
             raise ValueError("delta rule sizes must be positive, the key size at most 256")
         if num_heads % num_qk_heads:
             raise ValueError(f"num_heads {num_heads} is not a multiple of num_qk_heads {num_qk_heads}")
         self.hidden_size, self.num_heads, self.num_qk_heads = hidden_size, num_heads, num_qk_heads
         self.head_dim, self.value_dim, self.taps = head_dim, value_dim, taps
+        if gate_act not in ("sigmoid", "silu"):
+            raise ValueError(f"the gate is a sigmoid or silu, got {gate_act!r}")
         self.decay_rank, self.gate_rank, self.eps, self.unit_eps = decay_rank, gate_rank, float(eps), float(unit_eps)
+        self.gate_act = gate_act
         self.channels = 2 * num_qk_heads * head_dim + num_heads * value_dim
 
     def tensor_specs(self) -> dict[str, TensorSpec]:
         qk, vw, hd, h = self.num_qk_heads * self.head_dim, self.num_heads * self.value_dim, self.num_heads * self.head_dim, self.hidden_size
         conv = dict(init="normal", std=0.5)
-        return {
+        specs = {
             "q": TensorSpec((qk, h)), "k": TensorSpec((qk, h)), "v": TensorSpec((vw, h)),
             "q.conv": TensorSpec((qk, self.taps), **conv), "k.conv": TensorSpec((qk, self.taps), **conv),
             "v.conv": TensorSpec((vw, self.taps), **conv),
             "b": TensorSpec((self.num_heads, h)), "A_log": TensorSpec((self.num_heads,), init="normal", std=0.5),
-            "a1": TensorSpec((self.decay_rank, h)), "a2": TensorSpec((hd, self.decay_rank)),
-            "dt_bias": TensorSpec((hd,), init="normal", std=0.5),
-            "g1": TensorSpec((self.gate_rank, h)), "g2": TensorSpec((vw, self.gate_rank)),
             "norm": TensorSpec((self.value_dim,), init="one_plus_normal", std=0.05), "o": TensorSpec((h, vw)),
         }
+        if self.decay_rank is None:
+            specs["a"] = TensorSpec((self.num_heads, h))
+            specs["dt_bias"] = TensorSpec((self.num_heads,), init="normal", std=0.5)
+        else:
+            specs.update({"a1": TensorSpec((self.decay_rank, h)), "a2": TensorSpec((hd, self.decay_rank)),
+                          "dt_bias": TensorSpec((hd,), init="normal", std=0.5)})
+        if self.gate_rank is None:
+            specs["g"] = TensorSpec((vw, h))
+        else:
+            specs.update({"g1": TensorSpec((self.gate_rank, h)), "g2": TensorSpec((vw, self.gate_rank))})
+        return specs
 
     def load(self, tensors: Mapping[str, torch.Tensor], runtime: Runtime) -> None:
         self.runtime = runtime
-        self.in_proj = _padded([tensors[n] for n in ("q", "k", "v", "b", "a1", "g1")], runtime)
+        names = ("q", "k", "v", "b", "a" if self.decay_rank is None else "a1", "g" if self.gate_rank is None else "g1")
+        self.in_proj = _padded([tensors[n] for n in names], runtime)
         self.o_proj = Projection([tensors["o"]], None, runtime)
         self.conv_taps = torch.cat([runtime.place_vector_f32(tensors[f"{n}.conv"]) for n in ("q", "k", "v")], dim=0)
         self.a_log = runtime.place_vector_f32(tensors["A_log"])
         self.dt_bias = runtime.place_vector_f32(tensors["dt_bias"])
         # the second halves of the low-rank maps are applied inside the kernels, which read them transposed
-        self.a_up = runtime.place_matrix(tensors["a2"]).t().contiguous()
-        self.g_up = runtime.place_matrix(tensors["g2"]).t().contiguous()
+        self.a_up = None if self.decay_rank is None else runtime.place_matrix(tensors["a2"]).t().contiguous()
+        self.g_up = None if self.gate_rank is None else runtime.place_matrix(tensors["g2"]).t().contiguous()
         self.norm_weight = runtime.place_vector_f32(tensors["norm"])
 
     def cache_requirement(self):
@@ -136,10 +152,11 @@ class GatedDeltaRule(Mixer):
         proj = self.in_proj(x)
         beta_offset = self.channels
         low_offset = beta_offset + self.num_heads
-        gate_offset = low_offset + self.decay_rank
+        per_head = self.decay_rank is None
+        gate_offset = low_offset + (self.num_heads if per_head else self.decay_rank)
         q, k, v, g, beta = S.delta_prepare(
             proj, heads=self.num_heads, qk_heads=self.num_qk_heads, dim=self.head_dim, vdim=self.value_dim,
-            beta_offset=beta_offset, low_offset=low_offset, rank=self.decay_rank, taps=self.conv_taps,
+            beta_offset=beta_offset, low_offset=low_offset, rank=self.decay_rank or 0, taps=self.conv_taps,
             conv_state=cache.states["conv"], a_log=self.a_log, dt_bias=self.dt_bias, a_up=self.a_up, q_start=ctx.q_start,
             slots=ctx.slots, token_entry=ctx.token_entry, unit_eps=self.unit_eps, q_scale=self.head_dim ** -0.5,
         )
@@ -147,11 +164,64 @@ class GatedDeltaRule(Mixer):
             S.conv_state_update(proj, cache.states["conv"], ctx.q_start, ctx.slots)
         out = S.linear_scan(
             q, k, v, heads=self.num_heads, qk_heads=self.num_qk_heads, dim=self.head_dim, vdim=self.value_dim,
-            state=cache.states["state"], q_start=ctx.q_start, slots=ctx.slots, gate=g, beta=beta,
-            fixed_order=self.runtime.dtype == torch.float32,
+            state=cache.states["state"], q_start=ctx.q_start, slots=ctx.slots, gate=None if per_head else g,
+            row_decay=g if per_head else None, beta=beta, fixed_order=self.runtime.dtype == torch.float32,
         )
         gated = S.group_norm_gate(out, self.norm_weight, self.eps, proj, gate_offset=gate_offset, gate_up=self.g_up,
-                                  out_dtype=self.runtime.dtype)
+                                  act=self.gate_act, out_dtype=self.runtime.dtype)
+        return self.o_proj(gated, torch.float32)
+
+
+@MIXERS.register("retention")
+class Retention(Mixer):
+    """Retention (Sun et al.): linear attention with one constant decay per head behind a rotation.  ``q = W_q x``, ``k = W_k x``
+    (``heads x dim``), ``v = W_v x`` (``heads x vdim``); q and k are rotated by the position (``position``: a rotary encoding over the
+    leading columns of every head; ``None``: no rotation), k then times ``dim^(-1/2)``; per head ``S_t = decay_h S_(t-1) + k_t v_t^T``,
+    ``o_t = S_t^T q_t``.  Each head's ``o`` is divided by its root mean square (no weight); the heads side by side are multiplied with
+    ``silu(W_g x)``, then ``W_o``.  The rotated q and k stay float32 on their way into the recurrence.  The state ``[heads, dim, vdim]``
+    is float32, starts at zero and lives in the request's slot.  Tensors: ``q``, ``k``, ``v``, ``g`` (one stacked product), ``o``."""
+
+    graph_safe = True
+
+    def __init__(self, *, hidden_size: int, num_heads: int, head_dim: int, value_dim: int, decay: Sequence[float], eps: float,
+                 position: Mapping[str, Any] | None = None) -> None:
+        if min(hidden_size, num_heads, head_dim, value_dim) <= 0 or head_dim > 256:
+            raise ValueError("retention's sizes must be positive, the key size at most 256")
+        if len(decay) != num_heads:
+            raise ValueError(f"{len(decay)} decays for {num_heads} heads")
+        self.hidden_size, self.num_heads, self.head_dim, self.value_dim = hidden_size, num_heads, head_dim, value_dim
+        self.decay, self.eps = tuple(float(d) for d in decay), float(eps)
+        self.position = POSITION_ENCODINGS.build(position) if position else None
+
+    def children(self):
+        return (self.position,) if self.position is not None else ()
+
+    def tensor_specs(self) -> dict[str, TensorSpec]:
+        qk, vw, h = self.num_heads * self.head_dim, self.num_heads * self.value_dim, self.hidden_size
+        return {"q": TensorSpec((qk, h)), "k": TensorSpec((qk, h)), "v": TensorSpec((vw, h)), "g": TensorSpec((vw, h)),
+                "o": TensorSpec((h, vw))}
+
+    def load(self, tensors: Mapping[str, torch.Tensor], runtime: Runtime) -> None:
+        self.runtime = runtime
+        self.in_proj = _padded([tensors[n] for n in ("q", "k", "v", "g")], runtime)
+        self.o_proj = Projection([tensors["o"]], None, runtime)
+        self.decays = torch.tensor(self.decay, dtype=torch.float64).to(torch.float32).to(runtime.device)
+        if self.position is not None:
+            self.position.load({}, runtime)
+
+    def cache_requirement(self) -> FixedState:
+        return FixedState((self.num_heads, self.head_dim, self.value_dim), torch.float32)
+
+    def forward(self, x: torch.Tensor, ctx: Any, cache: Any) -> torch.Tensor:
+        proj = self.in_proj(x)                      # [N, q | k | v | g]
+        H, d, dv = self.num_heads, self.head_dim, self.value_dim
+        q, k = M.rotate_qk(proj, heads=H, head_dim=d, positions=ctx.positions, k_scale=d ** -0.5,
+                           rotary=self.position.rotary_layout() if self.position is not None else None)
+        out = S.linear_scan(
+            q, k, proj[:, 2 * H * d : H * (2 * d + dv)], heads=H, qk_heads=H, dim=d, vdim=dv, state=cache.state, q_start=ctx.q_start,
+            slots=ctx.slots, decay=self.decays, fixed_order=self.runtime.dtype == torch.float32,
+        )
+        gated = S.group_norm_gate(out, None, self.eps, proj, gate_offset=H * (2 * d + dv), group=dv, act="silu", out_dtype=self.runtime.dtype)
         return self.o_proj(gated, torch.float32)
 
 
@@ -324,7 +394,17 @@ class ParallelMixers(Mixer):
             return LayerCache(group=cache.group, tensors=cache.tensors, page_size=cache.page_size, states=states)
         return LayerCache(states=states)
 
-    def forward(self, x: torch.Tensor, ctx: Any, cache: Any) -> torch.Tensor:
+    @property
+    def returns_pieces(self) -> bool:
+        return len(self.branches) <= 2
+
+    def forward(self, x: torch.Tensor, ctx: Any, cache: Any, *, pieces: bool = False) -> "torch.Tensor | M.NormedBranches":
+        """``pieces``: return the branches' outputs unnormed, for a consumer that forms their mean itself (the norm behind this
+        part does)."""
+
+        if pieces and self.returns_pieces:
+            outs = [mixer.forward(x, ctx, self._branch_cache(name, mixer, cache)) for name, mixer in self.branches]
+            return M.NormedBranches(outs, self.out_weights, self.eps, 1.0 / len(self.branches))
         total = None
         for (name, mixer), weight in zip(self.branches, self.out_weights):
             out = mixer.forward(x, ctx, self._branch_cache(name, mixer, cache))

@@ -69,6 +69,9 @@ class LayerNorm(Norm):
         self.runtime = runtime
         self.weight = runtime.place_vector_f32(tensors["weight"])
 
+    def row_norm(self) -> tuple[torch.Tensor, float, bool]:
+        return self.weight, self.eps, True
+
     def add_norm(self, resid: torch.Tensor, delta: torch.Tensor | None, out_dtype: torch.dtype | None = None) -> torch.Tensor:
         return B.layer_norm(resid, delta, self.weight, self.eps, out_dtype or self.runtime.dtype)
 
