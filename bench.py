@@ -1498,6 +1498,189 @@ def _fumolorn_kernels(peak, timed) -> dict:
     return out
 
 
+# ------------------------------------------------------------------------------ Refolix beside Sorulix, Tafisun and Qwen3
+REFOLIX_EXPERTS, REFOLIX_TOP, REFOLIX_GROUPS, REFOLIX_KEEP = 8, 3, 4, 2
+
+
+def _refolix_config(width, ff, heads, kv_heads, d, pairs, vocab) -> dict:
+    """A parallel layer (capped window attention beside the delta rule) and a retention layer in turn; every token uses REFOLIX_TOP
+    of eight experts of ``ff / 4`` hidden units beside a shared unit of ``ff / 4``."""
+
+    moe = {"kind": "moe", "expert": {"ff": ff // 4},
+           "router": {"experts": REFOLIX_EXPERTS, "top": REFOLIX_TOP, "groups": {"count": REFOLIX_GROUPS, "keep": REFOLIX_KEEP}},
+           "shared": {"ff": ff // 4}}
+    parallel = {"type": "parallel", "mixer": {
+        "left": {"heads": heads, "kv_heads": kv_heads, "dim": d, "vdim": d, "scale": d ** -0.5, "softcap": 50.0, "mask": {"size": ROPULIX_WINDOW},
+                 "rot": {"base": 10000.0, "dims": d, "scaling": {"factor": 4.0, "original": 4096, "fast": 24.0, "slow": 2.0}}},
+        "right": {"heads": heads, "kv_heads": heads, "dim": d, "vdim": d, "conv": 4}}, "mlp": moe}
+    retention = {"type": "retention", "mixer": {"heads": heads, "dim": d, "vdim": d, "rot": {"base": 10000.0, "dims": d},
+                                                "decay": [1.0 - 2.0 ** (-5 - 3 * h / heads) for h in range(heads)]}, "mlp": moe}
+    return {"architecture": "Refolix", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "torch_dtype": "bfloat16", "postln_alpha": 2.0,
+            "logit_scale": 0.5, "logit_softcap": 25.0, "embedding": {"scale": width ** 0.5}, "layers": [parallel, retention] * pairs}
+
+
+def run_refolix(args) -> dict:
+    """Prefill and decode of Refolix at layer sizes of real models (random weights), beside Sorulix (the other design with softmax
+    attention beside a recurrence and with the delta rule), Tafisun (the other design with experts in groups and a gated shared one)
+    and Qwen3 at equal width, heads, head size and depth, through the same engine; then the new kernels alone against the bytes
+    or flops they must move, each beside the like kernel of an existing path."""
+
+    peak, timed, measure = _engine_measurer(args)
+    results = {}
+    for name in (() if args.only == "kernels" else args.size.split(",") if args.size else SORULIX_SIZES):
+        shape = SORULIX_SIZES[name]
+        results[name] = {"shape": dict(zip(("width", "ff", "heads", "kv_heads", "head_dim", "layer_pairs", "vocab"), shape)),
+                         "experts": REFOLIX_EXPERTS, "top": REFOLIX_TOP, "window": ROPULIX_WINDOW,
+                         "refolix": measure(_refolix_config(*shape), shape[-1])}
+        if args.only not in ("prefill", "decode"):
+            results[name]["sorulix_equal_size"] = measure(_sorulix_config(*shape), shape[-1])
+            results[name]["tafisun_equal_size"] = measure(_tafisun_config(*shape), shape[-1])
+            results[name]["qwen3_equal_size"] = measure(_qwen3_like(*shape), shape[-1])
+    kernels = _refolix_kernels(peak, timed) if args.only in ("all", "kernels") else {}
+    return {"workload": "refolix", "context": CONTEXT, "steps": args.steps, "warmup": max(args.warmup, 3), "dtype": "bfloat16",
+            "data": "synthetic token ids, seeded random weights", "peaks": peak, "models": results, "kernels": kernels}
+
+
+def _refolix_kernels(peak, timed) -> dict:
+    """Each new kernel alone at the 4k shape (width 4096, 32 heads of 128 over 8 key/value heads), replayed from a CUDA graph,
+    beside the kernel of an existing path that does the like work; fractions are of the measured copy bandwidth for the bytes a
+    kernel must move, or of the measured bf16 rate for its products."""
+
+    import torch
+    from types import SimpleNamespace
+
+    from llm_runtime_study_b200.ops import attention_rules
+    from llm_runtime_study_b200.ops import block_steps as B
+    from llm_runtime_study_b200.ops import functional as F
+    from llm_runtime_study_b200.ops import grouped as G
+    from llm_runtime_study_b200.ops import mixer_steps as M
+    from llm_runtime_study_b200.ops import sequence_state as S
+
+    dev = "cuda:0"
+    width, heads, kv_heads, d, page = 4096, 32, 8, 128, PAGE_SIZE
+    vw = heads * d
+    out = {}
+    cold = timed
+
+    def timed(fn, repeat):
+        fn()
+        fn()
+        torch.cuda.synchronize()
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph):
+            fn()
+        graph.replay()
+        return cold(graph.replay, repeat)
+
+    def beside(new, old, moved_new=None, moved_old=None, flops=None, flops_old=None):
+        """Microseconds of the new kernel and of the like one, and their fractions of the measured rates."""
+
+        t_new, t_old = timed(new, 20), timed(old, 20)
+        row = {"us": round(t_new * 1e3, 1), "like_us": round(t_old * 1e3, 1)}
+        if moved_new is not None:
+            row["of_measured_copy"] = [round(m / t / 1e6 / peak["hbm_gbs"], 3) for m, t in ((moved_new, t_new), (moved_old or moved_new, t_old))]
+        if flops is not None:
+            row["of_measured_bf16_burst"] = [round(f / t / 1e9 / peak["bf16_tflops"], 4) for f, t in ((flops, t_new), (flops_old or flops, t_old))]
+        return row
+
+    bf = lambda *shape: (0.05 * torch.randn(*shape, device=dev)).bfloat16()
+    f32 = lambda *shape: torch.randn(*shape, device=dev)
+    ints = lambda values: torch.tensor(values, dtype=torch.int32, device=dev)
+    inv_freq = torch.rand(d // 2, device=dev)
+    qw, kw = f32(d), f32(d)
+    # capped window attention (keys and values of equal and of different sizes) beside the chunked attention of equal reach
+    r1, r2 = torch.rand(heads, device=dev), torch.rand(heads, device=dev)
+    for seqs, length, new in ((1, 2048, 2048), (4, 2048, 2048), (8, 2048, 1), (32, 2048, 1)):
+        lengths, q_lens = [length] * seqs, [new] * seqs
+        pages = seqs * (length // page)
+        table = torch.arange(pages, dtype=torch.int32).view(seqs, -1).to(dev)
+        keys, values, narrow = bf(pages, kv_heads, page, d), bf(pages, kv_heads, page, d), bf(pages, kv_heads, page, d // 2)
+        q = bf(seqs * new, heads, d)
+        positions = ints([p for m, k in zip(lengths, q_lens) for p in range(m - k, m)])
+        entry = ints([i for i, k in enumerate(q_lens) for _ in range(k)])
+        ctx = SimpleNamespace(positions=positions, token_entry=entry, all_decode=new == 1, num_entries=seqs, q_lens=q_lens, kv_lens=lengths,
+                              max_kv_len=length, max_q_len=new, kv_len=ints(lengths))
+        cache, slim = (SimpleNamespace(keys=keys, values=v, page_size=page, group=0) for v in (values, narrow))
+        capped = lambda c: attention_rules.paged_attention_rules(q, c, ctx, table, scale=0.09, window=ROPULIX_WINDOW, softcap=50.0)
+        chunked = lambda: attention_rules.paged_attention_rules(q, cache, ctx, table, scale=0.09, chunk=TAFISUN_CHUNK, log_bias=(r1, r2))
+        seen = sum(min(p + 1, ROPULIX_WINDOW) for p in positions.tolist())
+        seen_chunk = sum(p % TAFISUN_CHUNK + 1 for p in positions.tolist())
+        name = f"attention_{seqs}x{length}_new_{new}"
+        row = kv_heads * 2 * d * 2
+        move = lambda keys_seen, bytes_row: None if new > 1 else keys_seen * bytes_row
+        out[name] = beside(lambda: capped(cache), chunked, move(seen, row), move(seen_chunk, row), 4.0 * heads * d * seen, 4.0 * heads * d * seen_chunk)
+        out[f"{name}_values_of_{d // 2}"] = beside(lambda: capped(slim), chunked, move(seen, row * 3 // 4), move(seen_chunk, row),
+                                                   3.0 * heads * d * seen, 4.0 * heads * d * seen_chunk)
+        if seqs != 4:      # what writes its q, k and v: norm, rotation and pages beside the norm and pages alone
+            n = seqs * new
+            rows = bf(n, (heads + 2 * kv_heads) * d)
+            write = lambda rotary: M.head_norm_write(rows, num_q_heads=heads, num_kv_heads=kv_heads, head_dim=d, value_dim=d, eps=1e-6, q_weight=qw,
+                                                     k_weight=kw, positions=positions, token_entry=entry, block_table=table, page_size=page,
+                                                     k_pool=keys, v_pool=values, rotary=rotary)
+            out[f"norm_rotate_write_{n}_tokens"] = beside(lambda: write((inv_freq, d, True, 1.1)), lambda: write(None), n * rows.shape[1] * 4)
+    # the scans: retention and the delta rule with one decay per head beside the constant decay on 16-bit rows and the channels' decays
+    for n, entries in ((2048, 1), (8, 8), (64, 64)):
+        proj = bf(n, 4 * vw)
+        q, k, v = (proj[:, i * vw : (i + 1) * vw] for i in range(3))
+        q32, k32, v32 = f32(n, vw), f32(n, vw), f32(n, vw)
+        state = torch.zeros(entries + 1, heads, d, d, device=dev)
+        q_start, slots = ints(list(range(0, n + 1, n // entries))), ints(list(range(entries)))
+        entry, positions = ints([e for e in range(entries) for _ in range(n // entries)]), ints([j for _ in range(entries) for j in range(n // entries)])
+        const, row_decay = torch.full((heads,), 0.97, device=dev), 0.9 + 0.1 * torch.rand(n, heads, device=dev)
+        gate, beta = 0.9 + 0.1 * torch.rand(n, vw, device=dev), torch.rand(n, heads, device=dev)
+        states = 2.0 * entries * heads * d * d * 4
+        sizes = dict(heads=heads, qk_heads=heads, dim=d, vdim=d, state=state, q_start=q_start, slots=slots)
+        name = f"{n}_tokens_{entries}_requests"
+        out[f"scan_retention_{name}"] = beside(
+            lambda: S.linear_scan(q32, k32, v, **sizes, decay=const), lambda: S.linear_scan(q, k, v, **sizes, decay=const),
+            states + n * vw * 14, states + n * vw * 10)
+        out[f"scan_delta_head_decay_{name}"] = beside(
+            lambda: S.linear_scan(q32, k32, v32, **sizes, row_decay=row_decay, beta=beta),
+            lambda: S.linear_scan(q32, k32, v32, **sizes, gate=gate, beta=beta), states + n * vw * 16, states + n * vw * 20)
+        # what they read: rotation, and the delta rule's preparation beside the one with a low-rank decay
+        taps, conv = f32(3 * vw, 4), torch.zeros(entries + 1, 3, 3 * vw, device=dev)
+        head_bias, bias, up = f32(heads), f32(vw), bf(d // 4, vw)
+        delta_proj = bf(n, 3 * vw + 2 * heads + vw)
+        prepare = lambda rank, a_up, dt: S.delta_prepare(
+            delta_proj, heads=heads, qk_heads=heads, dim=d, vdim=d, beta_offset=3 * vw, low_offset=3 * vw + heads, rank=rank, taps=taps,
+            conv_state=conv, a_log=head_bias, dt_bias=dt, a_up=a_up, q_start=q_start, slots=slots, token_entry=entry, unit_eps=1e-6, q_scale=0.1)
+        if entries != 8:
+            out[f"delta_prepare_{n}_tokens"] = beside(lambda: prepare(0, None, head_bias), lambda: prepare(d // 4, up, bias), n * vw * 18, n * vw * 22)
+            turned = torch.empty(n, vw, dtype=torch.bfloat16, device=dev)
+            out[f"rotate_qk_{n}_tokens"] = beside(
+                lambda: M.rotate_qk(proj, heads=heads, head_dim=d, positions=positions, k_scale=0.1, rotary=(inv_freq, d, False, 1.0)),
+                lambda: M.rope_slice(proj, turned, heads=heads, src_head=d, src_offset=0, dst_head=d, dst_offset=0, rot=d, rot_dims=d,
+                                     inv_freq=inv_freq, positions=positions), n * vw * 12, n * vw * 4)
+            x, w = f32(n, vw), f32(d)
+            out[f"read_out_{n}_tokens"] = beside(
+                lambda: S.group_norm_gate(x, None, 1e-6, proj, gate_offset=3 * vw, group=d, act="silu", out_dtype=torch.bfloat16),
+                lambda: S.group_norm_gate(x, w, 1e-6, proj, gate_offset=3 * vw, out_dtype=torch.bfloat16), n * vw * 8)
+    # the norm behind the sum in its three forms beside the norm on a sublayer's output; the router; the logits' scale and cap
+    outputs = REFOLIX_EXPERTS
+    router, correction, norm_w, scale = f32(outputs + 1, width), f32(outputs) * 0.1, f32(width), f32(width)
+    for n in (2048, 32):
+        x = bf(n, width)
+        wide = G.wide_tiles_pay(n, REFOLIX_TOP, x.dtype, width, 12288 // 4)
+        common = dict(top=REFOLIX_TOP, wide_tiles=wide, correction=correction, groups=REFOLIX_GROUPS, keep=REFOLIX_KEEP, extra=1)
+        new = lambda: G.route(x, router, None, score="sigmoid_all", group_best=2, renormalise=True, **common)
+        out[f"route_and_sort_{n}_tokens"] = beside(new, lambda: G.route(x, router, None, score="softmax_all", **common), n * width * 2)
+        routing = new()
+        rows, resid, left, right, shared = f32(routing.rows, width), f32(n, width), f32(n, width), f32(n, width), f32(n, width)
+        behind = lambda y: B.sum_norm(resid, y, norm_w, 1e-6, alpha=2.0, scale=scale, rounded_dtype=torch.bfloat16)
+        on_output = lambda y: M.norm_accumulate_round(y, norm_w, 1e-6, resid, torch.bfloat16)
+        pieces = M.PairedRows(rows, routing.pair_row, routing.weights, shared, routing.extra)
+        out[f"sum_norm_{n}_rows"] = beside(lambda: behind(left), lambda: on_output(left), n * width * 14)
+        out[f"sum_norm_experts_{n}_rows"] = beside(lambda: behind(pieces), lambda: on_output(M.PairedRows(rows, routing.pair_row, routing.weights)),
+                                                   n * width * (14 + 4 * REFOLIX_TOP), n * width * (10 + 4 * REFOLIX_TOP))
+        out[f"sum_norm_branches_{n}_rows"] = beside(
+            lambda: behind(M.NormedBranches([left, right], [norm_w, scale], 1e-6, 0.5)),
+            lambda: F.rmsnorm_accumulate(right, scale, 1e-6, 0.5, F.rmsnorm_accumulate(left, norm_w, 1e-6, 0.5)), n * width * 18, n * width * 20)
+    for n in (1, 32):
+        logits = f32(n, 151936)
+        out[f"logit_scale_and_cap_{n}_rows"] = beside(lambda: F.soft_cap(logits, 25.0, 0.5), lambda: F.soft_cap(logits, 25.0), n * 151936 * 8)
+    return out
+
+
 def run_reference(args) -> dict:
     """The unmodified reference from baseline/_ref: its own Qwen3ForCausalLM, paged cache,
     CUDA-graph decode and BatchScheduler, driven through Engine.create_scheduler()."""
@@ -1601,14 +1784,15 @@ def main() -> int:
     parser.add_argument("--batch", type=int, default=8)
     parser.add_argument("--context", type=int, default=0, help="with --only decode: cached tokens per request (default 2048)")
     parser.add_argument("--layers", type=int, default=0, help="fewer layers than the configuration has (named in config)")
-    parser.add_argument("--workload", choices=("default", "staggered14b", "decode32b", "sorulix", "ropulix", "mabedra", "tafisun", "fumolorn"), default="default",
+    parser.add_argument("--workload", choices=("default", "staggered14b", "decode32b", "sorulix", "ropulix", "mabedra", "tafisun", "fumolorn", "refolix"), default="default",
                         help="default: Qwen3-8B decode/prefill; staggered14b, decode32b: the larger configurations (either --impl); "
                              "sorulix: the Sorulix design beside Qwen3 at equal sizes, and its kernels alone; "
                              "ropulix: the Ropulix design beside Sorulix and Qwen3 at equal sizes, and its kernels alone; "
                              "mabedra: the Mabedra design beside Qwen3 and Ropulix at equal sizes, and its kernels alone; "
                              "tafisun: the Tafisun design beside Ropulix and Qwen3 at equal sizes, and its kernels alone; "
-                             "fumolorn: the Fumolorn design beside Ropulix, Sorulix and Qwen3 at equal sizes, and its kernels alone")
-    parser.add_argument("--size", default="", help="with --workload sorulix, ropulix, mabedra, tafisun or fumolorn: sizes to run, with commas (2k, 4k; default both)")
+                             "fumolorn: the Fumolorn design beside Ropulix, Sorulix and Qwen3 at equal sizes, and its kernels alone; "
+                             "refolix: the Refolix design beside Sorulix, Tafisun and Qwen3 at equal sizes, and its kernels alone")
+    parser.add_argument("--size", default="", help="with --workload sorulix, ropulix, mabedra, tafisun, fumolorn or refolix: sizes to run, with commas (2k, 4k; default both)")
     parser.add_argument("--only", choices=("all", "decode", "prefill", "kernels", "models"), default="all",
                         help="run only the decode steps or only the prefill (for profiler captures of a small case); "
                              "with --workload sorulix: only the kernels alone, or only the whole models")
@@ -1645,6 +1829,11 @@ def main() -> int:
             result = _unavailable("the reference has no model of this design")
         else:
             result = run_fumolorn(args)
+    elif args.workload == "refolix":
+        if args.impl == "reference":
+            result = _unavailable("the reference has no model of this design")
+        else:
+            result = run_refolix(args)
     else:
         result = run_reference(args) if args.impl == "reference" else run_ours(args)
     print(json.dumps(result))

@@ -613,3 +613,106 @@ def make_fumolorn_dir(path: Path, config: dict, seed: int, *, torch_dtype: str =
     (path / "config.json").write_text(json.dumps(config, indent=1), encoding="utf-8")
     write_file(path / "model.safetensors", state)
     return path, state
+
+
+# ----------------------------------------------------------------- Refolix
+def _refolix_moe(experts, top, ff, groups, shared):
+    return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top, "groups": {"count": groups[0], "keep": groups[1]}},
+            "shared": {"ff": shared} if shared else None}
+
+
+# A: sizes that are no multiples of 16, values wider and narrower than keys, one key/value head for three query heads, rotations
+# over part of a head and over all of it, frequencies stretched so that some pairs keep theirs, some are divided and some lie
+# between, a cap low enough to bite, a window of 5 beside pages of 4, convolutions of 4 taps and of 2, decays from fast to none,
+# experts in three groups of which two are kept, a layer without a feed-forward.
+REFOLIX_A = {
+    "architecture": "Refolix", "vocab": 211, "width": 64, "norm": {"eps": 1e-5}, "postln_alpha": 1.7, "logit_scale": 0.8, "logit_softcap": 3.0,
+    "embedding": {"scale": 2.5},
+    "layers": [
+        {"type": "parallel", "mixer": {
+            "left": {"heads": 3, "kv_heads": 1, "dim": 24, "vdim": 20, "scale": 0.4, "softcap": 2.0, "mask": {"size": 5},
+                     "rot": {"base": 500.0, "dims": 12, "scaling": {"factor": 4.0, "original": 64, "fast": 8.0, "slow": 1.0}}},
+            "right": {"heads": 6, "kv_heads": 2, "dim": 12, "vdim": 10, "conv": 4}},
+         "mlp": _refolix_moe(9, 3, 24, (3, 2), 40)},
+        {"type": "retention", "mixer": {"heads": 3, "dim": 20, "vdim": 12, "decay": [0.5, 0.97, 1.0], "rot": {"base": 100.0, "dims": 8}}, "mlp": None},
+        {"type": "retention", "mixer": {"heads": 1, "dim": 14, "vdim": 40, "decay": [0.995], "rot": {"base": 3000.0, "dims": 14}},
+         "mlp": _refolix_moe(6, 2, 40, (2, 1), 24)},
+        {"type": "parallel", "mixer": {
+            "left": {"heads": 2, "kv_heads": 2, "dim": 10, "vdim": 16, "scale": 0.3, "softcap": 30.0, "mask": {"size": 33},
+                     "rot": {"base": 10000.0, "dims": 10, "scaling": {"factor": 2.0, "original": 4096, "fast": 32.0, "slow": 1.0}}},
+            "right": {"heads": 2, "kv_heads": 1, "dim": 24, "vdim": 36, "conv": 2}},
+         "mlp": _refolix_moe(8, 8, 16, (4, 4), 16)},
+    ],
+}
+# B: every factor 1 (embedding, logits, the stream inside a norm), convolutions of one tap, a window of one position, groups of one
+# expert, a single expert used, a width that no vector divides, no shared expert in one layer, no cap on the logits.
+REFOLIX_B = {
+    "architecture": "Refolix", "vocab": 131, "width": 50, "norm": {"eps": 1e-6}, "postln_alpha": 1.0, "logit_scale": 1.0, "logit_softcap": None,
+    "embedding": {"scale": 1.0},
+    "layers": [
+        {"type": "retention", "mixer": {"heads": 2, "dim": 9, "vdim": 7, "decay": [0.9, 0.999], "rot": {"base": 10000.0, "dims": 2}},
+         "mlp": _refolix_moe(5, 1, 33, (5, 2), 9)},
+        {"type": "parallel", "mixer": {
+            "left": {"heads": 1, "kv_heads": 1, "dim": 8, "vdim": 40, "scale": 1.0, "softcap": 5.0, "mask": {"size": 1},
+                     "rot": {"base": 20.0, "dims": 4, "scaling": {"factor": 1.0, "original": 16, "fast": 4.0, "slow": 4.0}}},
+            "right": {"heads": 1, "kv_heads": 1, "dim": 40, "vdim": 5, "conv": 1}},
+         "mlp": _refolix_moe(4, 2, 17, (1, 1), None)},
+    ],
+}
+# C: sizes in steps of 16 throughout, which is what the tensor-core kernels of the bfloat16 run type take: keys and values of
+# different sizes, of equal ones, windows of a page, of a tile of keys and longer than every sequence.
+REFOLIX_C = {
+    "architecture": "Refolix", "vocab": 152, "width": 128, "norm": {"eps": 1e-6}, "postln_alpha": 2.2, "logit_scale": 1.5, "logit_softcap": 20.0,
+    "embedding": {"scale": 7.0},
+    "layers": [
+        {"type": "parallel", "mixer": {
+            "left": {"heads": 4, "kv_heads": 2, "dim": 32, "vdim": 48, "scale": 0.2, "softcap": 6.0, "mask": {"size": 16},
+                     "rot": {"base": 5000.0, "dims": 16, "scaling": {"factor": 16.0, "original": 128, "fast": 16.0, "slow": 2.0}}},
+            "right": {"heads": 4, "kv_heads": 4, "dim": 32, "vdim": 64, "conv": 4}},
+         "mlp": _refolix_moe(12, 3, 32, (3, 1), 64)},
+        {"type": "retention", "mixer": {"heads": 4, "dim": 64, "vdim": 32, "decay": [0.75, 0.99, 0.998, 0.9995], "rot": {"base": 20000.0, "dims": 32}},
+         "mlp": _refolix_moe(8, 4, 64, (4, 2), 32)},
+        {"type": "parallel", "mixer": {
+            "left": {"heads": 6, "kv_heads": 1, "dim": 96, "vdim": 64, "scale": 0.1, "softcap": 15.0, "mask": {"size": 64},
+                     "rot": {"base": 10000.0, "dims": 96, "scaling": {"factor": 2.0, "original": 4096, "fast": 32.0, "slow": 1.0}}},
+            "right": {"heads": 2, "kv_heads": 1, "dim": 64, "vdim": 32, "conv": 3}},
+         "mlp": None},
+        {"type": "parallel", "mixer": {
+            "left": {"heads": 2, "kv_heads": 1, "dim": 64, "vdim": 64, "scale": 0.125, "softcap": 50.0, "mask": {"size": 4096},
+                     "rot": {"base": 1000.0, "dims": 64, "scaling": None}},
+            "right": {"heads": 3, "kv_heads": 1, "dim": 16, "vdim": 16, "conv": 5}},
+         "mlp": _refolix_moe(8, 2, 64, (2, 1), 64)},
+    ],
+}
+REFOLIX = {"A": (REFOLIX_A, 61, 4), "B": (REFOLIX_B, 62, 16), "C": (REFOLIX_C, 63, 16)}   # config, seed, page size
+
+
+def make_refolix_dir(path: Path, config: dict, seed: int, *, torch_dtype: str = "float32", gain: float = 6.0):
+    """Write a Refolix model folder with random weights; return (path, {name: CPU tensor as stored}).  The matrices are
+    drawn ``gain`` times larger than the framework's default, so that gates and scores are not all alike; the corrections are drawn
+    wide (many choice scores are negative) and the delta rule's decays slow enough for its state to outlive a portion."""
+
+    from llm_runtime_study_b200.config import RefolixConfig
+    from llm_runtime_study_b200.models.description import tensor_schema
+    from llm_runtime_study_b200.models.refolix import describe_refolix
+    from llm_runtime_study_b200.weights.random_init import random_state
+    from llm_runtime_study_b200.weights.safetensors_io import write_file
+
+    schema = tensor_schema(describe_refolix(RefolixConfig.from_dict(config)))
+    dtype = {"float32": torch.float32, "bfloat16": torch.bfloat16}[torch_dtype]
+    state = random_state(schema, seed, dtype=torch.float32, include_optional=False)
+    for name, tensor in state.items():
+        if name == "embed":
+            tensor *= 40.0
+        elif name.endswith(".correction"):
+            tensor *= 4.0
+            tensor -= 0.6
+        elif name.endswith(".dt_bias"):
+            tensor -= 3.0
+        elif tensor.dim() == 2 and not name.endswith((".router", ".sg", ".conv")):
+            tensor *= gain
+    state = {name: tensor.to(dtype) for name, tensor in state.items()}
+    path.mkdir(parents=True, exist_ok=True)
+    (path / "config.json").write_text(json.dumps(config, indent=1), encoding="utf-8")
+    write_file(path / "model.safetensors", state)
+    return path, state
