@@ -80,11 +80,9 @@ struct AttnParams {
 template <int NT>
 __device__ __forceinline__ void load_kv_tile(bf16* ks, bf16* vs, const AttnParams& p, const int* table,
                                              int kvh, int t0, int lo, int hi) {
-  // a row's chunks of 16 bytes: the first CH of them hold its key (and, of equal size, its value beside it), those behind
-  // them, where the sizes differ, its value
-  constexpr int CH = D / 8, CV = D == DV ? 0 : DV / 8;
-  for (int c = threadIdx.x; c < BN * (CH + CV); c += NT) {
-    const int r = c / (CH + CV), ch = c - r * (CH + CV);
+  constexpr int CK = D / 8, CV = DV / 8, CH = CK > CV ? CK : CV;      // chunks of 16 bytes in a row
+  for (int c = threadIdx.x; c < BN * CH; c += NT) {
+    const int r = c / CH, ch = c - r * CH;
     const int t = t0 + r;
     size_t row = 0;
     int bytes = 0;
@@ -97,15 +95,8 @@ __device__ __forceinline__ void load_kv_tile(bf16* ks, bf16* vs, const AttnParam
         bytes = 16;
       }
     }
-    if constexpr (CV == 0) {
-      const size_t off = bytes ? row * D + ch * 8 : 0;
-      cp_async_16(ks + r * LDS + ch * 8, p.k_pool + off, bytes);
-      cp_async_16(vs + r * LDV + ch * 8, p.v_pool + off, bytes);
-    } else if (ch < CH) {
-      cp_async_16(ks + r * LDS + ch * 8, p.k_pool + (bytes ? row * D + ch * 8 : 0), bytes);
-    } else {
-      cp_async_16(vs + r * LDV + (ch - CH) * 8, p.v_pool + (bytes ? row * DV + (ch - CH) * 8 : 0), bytes);
-    }
+    if (CK == CH || ch < CK) cp_async_16(ks + r * LDS + ch * 8, p.k_pool + (bytes ? row * D + ch * 8 : 0), bytes);
+    if (CV == CH || ch < CV) cp_async_16(vs + r * LDV + ch * 8, p.v_pool + (bytes ? row * DV + ch * 8 : 0), bytes);
   }
 }
 
@@ -384,11 +375,11 @@ __global__ void __launch_bounds__(128) decode_attention_kernel(AttnParams p) {
   const int nblocks = c1 >= c0 ? (c1 - c0) / WB + 1 : 0;  // 16-key blocks in this CTA's part
   const int hi_here[2] = {min(row_hi[0], c1), min(row_hi[1], c1)};
   auto load_block = [&](int block, int buf) {
-    constexpr int CH = D / 8, CV = D == DV ? 0 : DV / 8;       // as in load_kv_tile
+    constexpr int CK = D / 8, CV = DV / 8, CH = CK > CV ? CK : CV;
     const int t0 = c0 + block * WB;
 #pragma unroll
-    for (int c = lane; c < WB * (CH + CV); c += 32) {
-      const int r = c / (CH + CV), ch = c - r * (CH + CV);
+    for (int c = lane; c < WB * CH; c += 32) {
+      const int r = c / CH, ch = c - r * CH;
       const int t = t0 + r;
       size_t row = 0;
       int bytes = 0;
@@ -401,15 +392,8 @@ __global__ void __launch_bounds__(128) decode_attention_kernel(AttnParams p) {
           bytes = 16;
         }
       }
-      if constexpr (CV == 0) {
-        const size_t off = bytes ? row * D + ch * 8 : 0;
-        cp_async_16(wk + (buf * WB + r) * LDS + ch * 8, p.k_pool + off, bytes);
-        cp_async_16(wv + (buf * WB + r) * LDV + ch * 8, p.v_pool + off, bytes);
-      } else if (ch < CH) {
-        cp_async_16(wk + (buf * WB + r) * LDS + ch * 8, p.k_pool + (bytes ? row * D + ch * 8 : 0), bytes);
-      } else {
-        cp_async_16(wv + (buf * WB + r) * LDV + (ch - CH) * 8, p.v_pool + (bytes ? row * DV + (ch - CH) * 8 : 0), bytes);
-      }
+      if (CK == CH || ch < CK) cp_async_16(wk + (buf * WB + r) * LDS + ch * 8, p.k_pool + (bytes ? row * D + ch * 8 : 0), bytes);
+      if (CV == CH || ch < CV) cp_async_16(wv + (buf * WB + r) * LDV + ch * 8, p.v_pool + (bytes ? row * DV + ch * 8 : 0), bytes);
     }
   };
   if (warp < nblocks) {

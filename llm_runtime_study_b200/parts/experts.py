@@ -12,7 +12,7 @@ from ..ops import grouped as G
 from ..ops.mixer_steps import PairedRows
 from ..weights.checkpoint import TensorSpec
 from .base import FEED_FORWARDS, FeedForward, Runtime
-from .linear import Projection
+from .linear import Projection, interleaved_projection
 
 ACTS = ("relu2", "silu_glu", "limited_glu")
 GATED = ("silu_glu", "limited_glu")
@@ -120,7 +120,10 @@ class RoutedExperts(FeedForward):
         self.down = torch.stack([runtime.place_matrix(tensors[f"e{e}.down"]) for e in range(self.experts)])
         self.shared_up = self.shared_down = None
         if self.shared_size is not None:
-            self.shared_up = Projection([tensors["shared.gate"], tensors["shared.up"]], None, runtime)
+            gate, up = runtime.place_matrix(tensors["shared.gate"]), runtime.place_matrix(tensors["shared.up"])
+            # rows of gate and up in turn where the width allows: the projection's kernels then form the gated unit themselves
+            self.shared_interleaved = self.act == "silu_glu" and self.shared_size % 8 == 0
+            self.shared_up = interleaved_projection(gate, up, runtime) if self.shared_interleaved else Projection([gate, up], None, runtime)
             self.shared_down = Projection([tensors["shared.down"]], None, runtime)
 
     # the weighted sum over a token's experts may be left to the consumer (``PairedRows``): see ``forward``
@@ -173,4 +176,4 @@ class RoutedExperts(FeedForward):
     def _shared_hidden(self, x: torch.Tensor) -> torch.Tensor:
         if self.act == "limited_glu":
             return F.glu_limit(self.shared_up(x), self.shared_limit, self.alpha)
-        return B.silu_mul_scaled(self.shared_up(x))
+        return self.shared_up.swiglu(x) if self.shared_interleaved else B.silu_mul_scaled(self.shared_up(x))

@@ -144,3 +144,12 @@ class Projection:
         if self.bias is not None:
             y += self.bias.to(y.dtype)
         return y
+
+
+def interleaved_projection(gate: torch.Tensor, up: torch.Tensor, runtime: Runtime) -> Projection:
+    """One projection of gate and up features (``[I, K]`` each, placed) interleaved in blocks of eight, as ``Projection.swiglu`` takes
+    them; ``I`` is a multiple of eight."""
+
+    blocks = gate.shape[0] // 8
+    stacked = torch.stack((gate.view(blocks, 8, -1), up.view(blocks, 8, -1)), dim=1).reshape(2 * gate.shape[0], -1)
+    return Projection([stacked], None, runtime)

@@ -10,7 +10,7 @@ from ..ops import block_steps as B
 from ..ops import functional as F
 from ..weights.checkpoint import TensorSpec
 from .base import FEED_FORWARDS, FeedForward, Runtime
-from .linear import Projection
+from .linear import Projection, interleaved_projection
 
 
 @FEED_FORWARDS.register("swiglu")
@@ -44,14 +44,7 @@ class GatedMLP(FeedForward):
         # ([g0..g7, u0..u7, g8..g15, ...]): a projection kernel then holds matching gate and
         # up features in one tile and can apply SiLU * up before it writes anything.
         self.interleaved = self.intermediate_size % 8 == 0
-        if self.interleaved:
-            blocks = self.intermediate_size // 8
-            stacked = torch.stack((gate.view(blocks, 8, -1), up.view(blocks, 8, -1)), dim=1).reshape(2 * self.intermediate_size, -1)
-            del gate, up
-            self.gate_up_proj = Projection([stacked], None, runtime)
-            del stacked
-        else:
-            self.gate_up_proj = Projection([gate, up], None, runtime)
+        self.gate_up_proj = interleaved_projection(gate, up, runtime) if self.interleaved else Projection([gate, up], None, runtime)
         self.down_proj = Projection([tensors[self.names[2]]], None, runtime)
 
     adds_to_residual = True

@@ -716,3 +716,17 @@ def make_refolix_dir(path: Path, config: dict, seed: int, *, torch_dtype: str = 
     (path / "config.json").write_text(json.dumps(config, indent=1), encoding="utf-8")
     write_file(path / "model.safetensors", state)
     return path, state
+
+
+def rows_without_a_close_call(margins, tokens: int, close: float = 2e-2, undecided: float = 5e-3, reach: int = 8) -> torch.Tensor:
+    """Rows of a request that rounding alone cannot send to other experts: the token's own choices were decided by more than
+    ``close``, and none of the ``reach`` tokens before it, whose keys and states it reads, by less than ``undecided``.  ``margins``:
+    one list of ``tokens`` numbers per routed layer."""
+
+    if not margins:
+        return torch.ones(tokens, dtype=torch.bool)
+    least = torch.tensor(margins).min(dim=0).values
+    clear = least > close
+    for t in (least < undecided).nonzero().flatten().tolist():
+        clear[t : t + 1 + reach] = False
+    return clear

@@ -235,10 +235,11 @@ def route(z: torch.Tensor, correction: torch.Tensor, *, top: int, groups: int, k
     return chosen, w / (w.sum(dim=1, keepdim=True) + 1e-20)
 
 
-def gated_unit(h, gate, up, down, store=keep) -> torch.Tensor:
-    """``W_down (silu(W_gate h) * (W_up h))``."""
+def gated_unit(h, gate, up, down, store=keep, between=None) -> torch.Tensor:
+    """``W_down (silu(W_gate h) * (W_up h))``; ``between``: the rounding of the two products (default: ``store``)."""
 
-    return store(silu(store(h @ gate.T)) * store(h @ up.T)) @ down.T
+    between = between or store
+    return store(silu(between(h @ gate.T)) * between(h @ up.T)) @ down.T
 
 
 def moe(h, w: Mapping[str, torch.Tensor], mlp: Mapping, store=keep, margins: list | None = None) -> torch.Tensor:
@@ -251,7 +252,7 @@ def moe(h, w: Mapping[str, torch.Tensor], mlp: Mapping, store=keep, margins: lis
         if at.numel():
             out[at] += weights[at, place][:, None] * gated_unit(h[at], *(w[f"e{e}.{n}"] for n in ("gate", "up", "down")), store)
     if mlp.get("shared"):
-        out = out + sigmoid(h @ w["shared.sg"].T) * gated_unit(h, *(w[f"shared.{n}"] for n in ("gate", "up", "down")), store)
+        out = out + sigmoid(h @ w["shared.sg"].T) * gated_unit(h, *(w[f"shared.{n}"] for n in ("gate", "up", "down")), store, keep)
     return out
 
 

@@ -16,7 +16,6 @@ pytestmark = pytest.mark.gpu
 
 TOL32 = (3e-5, 2e-4)
 BF16_USUAL, BF16_WORST = 6e-2, 3e-1
-CLOSE_CALL = 2e-2
 
 
 def _moe(rng):
@@ -80,7 +79,7 @@ def test_random_configuration(case, dtype, tmp_path):
     for rid, tokens in requests.items():
         margins = []
         expected[rid] = plain.forward(raw, weights, tokens, store=store, margins=margins)
-        clear[rid] = torch.tensor(margins).min(dim=0).values > CLOSE_CALL if margins else torch.ones(len(tokens), dtype=torch.bool)
+        clear[rid] = helpers.rows_without_a_close_call(margins, len(tokens))
     loaded = load(path, device="cuda:0", dtype=dtype, strict_dtype=False)
     traces = {
         "whole": helpers.trace_whole(requests),
