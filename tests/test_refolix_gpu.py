@@ -444,7 +444,7 @@ def test_a_token_kept_over_two_thousand_others(dtype):
         q[:, h * dim] = 1.0
         v[:, h * vdim :(h + 1) * vdim] = 100.0
         v[2, h * vdim :(h + 1) * vdim] = torch.arange(1.0, vdim + 1)
-    decay = dev(torch.tensor([1.0, 0.9990234375]))
+    decay = dev(torch.tensor([1.0, 0.99853515625]))
     state = torch.zeros(1, 2, dim, vdim, device=DEV)
     out = []
     for a, b in ((0, 1000), (1000, 2001), (2001, 2002), (2002, 2003)):
@@ -454,7 +454,7 @@ def test_a_token_kept_over_two_thousand_others(dtype):
     value = torch.arange(1.0, vdim + 1, dtype=torch.float64)
     for p in (2, 3, 999, 1000, 2000, 2001, 2002):
         close(out[p, :vdim], value, 1e-6)
-        close(out[p, vdim:], value * 0.9990234375 ** (p - 2), 1e-4)
+        close(out[p, vdim:], value * 0.99853515625 ** (p - 2), 1e-4)
 
 
 # ----------------------------------------------------------------------------------------------- experts
